@@ -19,8 +19,8 @@ LIB_PATH = os.path.join(os.path.dirname(_HERE), "libb200nn.so")
 
 OK, ERR_SHAPE, ERR_DIM, ERR_UNSUPPORTED, ERR_CUDA, ERR_DEVICE, ERR_ARG, ERR_IO, ERR_MISSING = range(9)
 ACT_NONE, ACT_GELU_TANH, ACT_GELU_SIGMOID, ACT_RELU, ACT_SILU, ACT_SIGMOID = range(6)
-GELU_SIGMOID, QUANT_LM_HEAD, ARGMAX_LAST, STOP_ON_EOS, TOKENS_ONLY, WEIGHTS_OUT_IN = 1, 2, 4, 8, 16, 32
-PROF_NAMES = ("embed", "layernorm", "linear", "attention", "lm_head", "argmax")
+GELU_SIGMOID, QUANT_LM_HEAD, ARGMAX_LAST, STOP_ON_EOS, TOKENS_ONLY, WEIGHTS_OUT_IN, LM_F32 = 1, 2, 4, 8, 16, 32, 64
+PROF_NAMES = ("embed", "layernorm", "linear", "attention", "lm_head", "argmax", "recurrence")
 
 _KINDS = {ERR_SHAPE: "ShapeMismatch", ERR_DIM: "DimOutOfRange", ERR_UNSUPPORTED: "KernelNotFound",
           ERR_CUDA: "Cuda", ERR_DEVICE: "DeviceTimeout", ERR_ARG: "InvalidArgument", ERR_IO: "Io",
@@ -61,6 +61,10 @@ class _Diag(C.Structure):
                 ("final_block_last", C.c_float * 4), ("block0_nonfinite", C.c_int32), ("final_block_nonfinite", C.c_int32),
                 ("ln_f_last", C.c_float * 4), ("top_tokens", C.c_uint32 * 5), ("top_scores", C.c_float * 5),
                 ("n_top", C.c_int32)]
+
+
+class _LmInfo(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("n_layer", "width", "vocab_size", "n_positions", "eos_token")]
 
 
 class _Weights(C.Structure):
@@ -179,6 +183,16 @@ def load_library() -> C.CDLL:
             "b200nn_safetensors_read": (i32, [vp, i32, vp, sz]),
             "b200nn_safetensors_last_error": (C.c_char_p, []),
             "b200nn_gpt2_load_safetensors": (i32, [vp, C.c_char_p, C.POINTER(_Cfg), sz, u32, vpp]),
+            "b200nn_lm_create": (i32, [vp, C.c_char_p, sz, C.POINTER(C.c_char_p), C.POINTER(_f32p), szp, u32, vpp]),
+            "b200nn_lm_load": (i32, [vp, C.c_char_p, u32, vpp]), "b200nn_gpt2_as_lm": (vp, [vp]),
+            "b200nn_lm_destroy": (None, [vp]), "b200nn_lm_get_info": (i32, [vp, C.POINTER(_LmInfo)]),
+            "b200nn_lm_family": (C.c_char_p, [vp]),
+            "b200nn_lm_cache_create": (i32, [vp, sz, sz, vpp]), "b200nn_lm_session_create": (i32, [vp, sz, sz, u32, vpp]),
+            "b200nn_lm_generate_batch": (i32, [vp, _u32p, sz, sz, sz, u32, _u32p, szp]),
+            "b200nn_lm_generate_sampling": (i32, [vp, _u32p, sz, sz, sz, C.c_float, C.POINTER(C.c_uint64), _u32p, szp]),
+            "b200nn_kvcache_acquire": (i32, [vp, C.POINTER(i32)]), "b200nn_kvcache_release": (i32, [vp, i32]),
+            "b200nn_kvcache_slot_len": (sz, [vp, i32]),
+            "b200nn_lm_step": (i32, [vp, sz, C.POINTER(i32), szp, _u32p, sz, szp, _f32p]),
             "b200nn_bpe_load": (i32, [C.c_char_p, u32, vpp]),
             "b200nn_bpe_create": (i32, [C.c_char_p, szp, _u32p, sz, u32, vpp]),
             "b200nn_bpe_destroy": (None, [vp]), "b200nn_bpe_vocab_size": (sz, [vp]),
@@ -397,3 +411,4 @@ from .tokenizer import Gpt2Tokenizer, TokenizerError, GPT2_VOCAB_SIZE, ENDOFTEXT
 from .checkpoint import (SafeTensorsFile, TensorInfo, list_tensors, load_all_tensors, load_gpt2_weights,  # noqa: E402
                          load_int4_tensors, TensorData, WeightMapping, LoadedWeights, map_weight, map_weight_t,
                          load_safetensors_raw, load_safetensors_mapped, load_safetensors, gpt2_weight_map)
+from .lm import LanguageModel, RequestBatch, load_model  # noqa: E402

@@ -90,7 +90,7 @@ class KvCache:
         self.model = model
         self.h = C.c_void_p()
         cap = capacity or model.config.n_positions
-        model.reg.check(model.reg.lib.b200nn_kvcache_create(model.h, batch, cap, C.byref(self.h)))
+        model.reg.check(model.reg.lib.b200nn_lm_cache_create(model.lm_handle(), batch, cap, C.byref(self.h)))
 
     def len(self):
         return int(self.model.reg.lib.b200nn_kvcache_len(self.h))
@@ -291,6 +291,12 @@ class Gpt2Model:
             out.ctypes.data_as(_u32p), lens))
         return out, np.array(list(lens), dtype=np.int64)
 
+    vocab_size = property(lambda self: self.config.vocab_size)
+
+    def lm_handle(self):
+        """This model as the family-independent handle (``LanguageModel``'s)."""
+        return C.c_void_p(self.reg.lib.b200nn_gpt2_as_lm(self.h))
+
     def quantized_memory_bytes(self):
         return int(self.reg.lib.b200nn_gpt2_quantized_memory_bytes(self.h))
 
@@ -329,7 +335,7 @@ class DecodeSession:
     def __init__(self, model: Gpt2Model, batch: int, capacity: int, flags: int = 0):
         self.model, self.reg, self.batch, self.capacity = model, model.reg, batch, capacity
         self.h = C.c_void_p()
-        self.reg.check(self.reg.lib.b200nn_session_create(model.h, batch, capacity, model.flags | flags, C.byref(self.h)))
+        self.reg.check(self.reg.lib.b200nn_lm_session_create(model.lm_handle(), batch, capacity, model.flags | flags, C.byref(self.h)))
 
     def prefill(self, prompts):
         p = np.ascontiguousarray(prompts, dtype=np.uint32)

@@ -93,6 +93,7 @@ int block_run(b200nn_block *b, const b200nn_tensor *x, const float *cached_k, co
     kv.m = m;
     kv.batch = 1;
     kv.cap = cap;
+    kv.n_head = H;
     kv.len = past;
     TRY(dev_alloc(ctx, H * cap * 64 * sizeof(__half), &kv.k));
     TRY(dev_alloc(ctx, H * cap * 64 * sizeof(__half), &kv.v));

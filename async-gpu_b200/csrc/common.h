@@ -1,6 +1,7 @@
 // Internal declarations shared by the translation units of libb200nn.
 #pragma once
 
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
 
@@ -74,6 +75,7 @@ struct b200nn_ctx {
     int tc_persistent = 1;        // the plain fp16 GEMM runs one persistent block per SM from two 256-row tiles per SM on
     int int4_via_f16 = 1;         // int4 Linears with that many tiles dequantise the weight to fp16 once and use that GEMM
     std::shared_ptr<DevBuf> wh;   // the dequantised weight, [N,K] fp16, one Linear at a time
+    int lm_portion = 0;           // hybrid models: most new tokens of one sequence in a pass (0 = 2048); read when a cache is created
     bool capturing = false;      // true while a decode step is being captured into a graph
     // one persistent kernel for all transformer blocks of an int4 decode step (decode_persistent.cu)
     int persist = 0;              // 1: decode steps of persist_min_rows..persist_max_rows rows take it (opt-in: measured
@@ -205,23 +207,48 @@ int int4_weight_ln_fold(b200nn_ctx *ctx, const Int4Weight &w, const float *g_dev
 // f32 weight of a Linear, stored [K,N] (= [in,out]) row-major on the device.
 // w_nk_h: the same weight rounded to fp16 and stored [N,K] (K contiguous), the operand of the
 // tensor-core GEMM that serves more than four rows; absent when a value does not fit fp16's range.
+// exact: the f32 FMA kernels serve every row count (no 16-bit representation is made).
 struct F32Weight {
     int K = 0, N = 0;
+    bool exact = false;
     std::shared_ptr<DevBuf> w_kn, bias, w_nk_h;
 };
 // weight given as [out,in] (Linear layout) or [in,out] (checkpoint layout)
 int f32_weight_upload(b200nn_ctx *ctx, const float *w, bool is_out_in, const float *bias, size_t K, size_t N,
-                      F32Weight *out);
+                      F32Weight *out, bool exact = false);
+
+// bfloat16 weight of a Linear, stored [N,K] (K contiguous, a multiple of 8): the operand of the tensor-core
+// GEMM, which serves it for every row count.  With groups > 1 the Linear is block diagonal: output group g
+// (group_n features, group_stride columns apart in the output) is the product of weight rows
+// [g * tiles * 128, ...) and the K activation columns that start at g * group_kx; a group's rows are
+// padded with zeros to whole 128-feature tiles.
+struct B16Weight {
+    int K = 0, N = 0;
+    int groups = 1, group_n = 0, group_tiles = 0, group_kx = 0, group_stride = 0;
+    std::shared_ptr<DevBuf> w_nk;
+};
+int b16_weight_upload(b200nn_ctx *ctx, const float *w_nk, size_t K, size_t N, B16Weight *out);
+int b16_grouped_weight_upload(b200nn_ctx *ctx, const float *w_gnk, size_t groups, size_t Ng, size_t Kg, size_t x_stride,
+                              size_t out_stride, B16Weight *out);
 
 // ---------------------------------------------------------------------------------------------
 // epilogue shared by every Linear kernel
 // ---------------------------------------------------------------------------------------------
-enum { EPI_STORE = 0, EPI_RESID = 1, EPI_QKV = 2, EPI_RESID_LN = 3 };
+enum { EPI_STORE = 0, EPI_RESID = 1, EPI_QKV = 2, EPI_RESID_LN = 3, EPI_GLU = 4, EPI_ROPE = 5 };
+enum { OUT_F32 = 0, OUT_F16 = 1, OUT_BF16 = 2 };
+
+// Where the token rows of a pass sit: row r is position pos[r * pos_stride] of the sequence in cache slot
+// slot[r] (null: slot r).  pos_stride 0: one position for all rows (lockstep decoding).
+struct RowMap {
+    const int *pos = nullptr;
+    int pos_stride = 0;
+    const int *slot = nullptr;
+};
 
 struct Epilogue {
     int mode = EPI_STORE;
     int act = B200NN_ACT_NONE;
-    int out_half = 0;          // out is __half* instead of float*
+    int out_half = 0;          // element type of out: OUT_F32, OUT_F16 or OUT_BF16
     const float *bias = nullptr;
     void *out = nullptr;       // [M, ldo]
     int ldo = 0;
@@ -254,6 +281,17 @@ struct Epilogue {
     __half *xg_out = nullptr;
     const float *next_g = nullptr;
     float *stats_out = nullptr;
+    // EPI_GLU: the weight rows come in groups of four (two gates, then the two matching up projections);
+    // features n..n+3 give out[m, n/2 .. n/2+1] = act(gate) * up, with ldo the width of the product.
+    // EPI_ROPE: the features are heads of rope_head columns, whose columns rope_at .. rope_at + 2 rope_pairs
+    // are adjacent (u, v) pairs rotated by the angle table rope_tab [position][pair] (cos, sin) before they
+    // are stored; the row's position comes from rows.
+    int rope_head = 0, rope_at = 0, rope_pairs = 0;
+    const float2 *rope_tab = nullptr;
+    RowMap rows;
+    // row_scale: finished values are multiplied by row_scale[m * rs_ld + n / rs_cols] (a per-head gate)
+    const float *row_scale = nullptr;
+    int rs_ld = 0, rs_cols = 1;
 };
 
 // ---------------------------------------------------------------------------------------------
@@ -268,6 +306,8 @@ int launch_int4_gemm_tc(b200nn_ctx *ctx, const Int4Weight &w, const __half *x, i
 int launch_f32_linear(b200nn_ctx *ctx, const F32Weight &w, const void *x, bool x_half, int M, const Epilogue &epi);
 bool f16_gemm_tc_supported(const b200nn_ctx *ctx, const F32Weight &w, int M);
 int launch_f16_gemm_tc(b200nn_ctx *ctx, const F32Weight &w, const __half *x, int M, const Epilogue &epi);
+// x: bf16 [M, ldx] (ldx >= the activation columns the weight reads, a multiple of 8)
+int launch_b16_linear(b200nn_ctx *ctx, const B16Weight &w, const __nv_bfloat16 *x, int ldx, int M, const Epilogue &epi);
 bool int4_via_f16_supported(const b200nn_ctx *ctx, const Int4Weight &w, int M);
 int launch_int4_via_f16(b200nn_ctx *ctx, const Int4Weight &w, const __half *x, int M, const Epilogue &epi);
 

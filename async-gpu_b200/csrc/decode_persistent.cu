@@ -837,7 +837,7 @@ bool decode_persistent_supported(const b200nn_gpt2 *m, int rows) {
 }
 
 int decode_persistent_prepare(b200nn_session *s) {
-    b200nn_gpt2 *m = s->m;
+    b200nn_gpt2 *m = s->gpt2;
     b200nn_ctx *ctx = m->ctx;
     const size_t B = s->batch, d = m->cfg.n_embd, L = m->cfg.n_layer;
     std::vector<pd::Layer> h(L);
@@ -868,7 +868,7 @@ int decode_persistent_prepare(b200nn_session *s) {
 }
 
 int launch_decode_layers(b200nn_session *s, bool profile) {
-    b200nn_gpt2 *m = s->m;
+    b200nn_gpt2 *m = s->gpt2;
     b200nn_ctx *ctx = m->ctx;
     const int B = (int)s->batch, d = m->cfg.n_embd, H = m->cfg.n_head;
     static bool attr_done[16] = {};

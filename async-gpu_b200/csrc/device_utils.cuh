@@ -35,6 +35,20 @@ __device__ __forceinline__ float apply_act(float v, int act) {
     }
 }
 
+__device__ __forceinline__ uint32_t pack_bf16x2(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t *>(&h);
+}
+__device__ __forceinline__ uint32_t pack_f16x2(float a, float b) {
+    const __half2 h = __floats2half2_rn(a, b);
+    return *reinterpret_cast<const uint32_t *>(&h);
+}
+__device__ __forceinline__ uint32_t epi_pack2(const Epilogue &e, float a, float b) {
+    return e.out_half == OUT_BF16 ? pack_bf16x2(a, b) : pack_f16x2(a, b);
+}
+__device__ __forceinline__ int row_pos(const RowMap &r, int m) { return r.pos[(size_t)m * r.pos_stride]; }
+__device__ __forceinline__ int row_slot(const RowMap &r, int m) { return r.slot ? r.slot[m] : m; }
+
 // Consumes one finished output value v (bias already added) for row m (token), column n (feature).
 __device__ __forceinline__ void epi_store(const Epilogue &e, int m, int n, float v) {
     if (e.no_store) return;
@@ -57,8 +71,11 @@ __device__ __forceinline__ void epi_store(const Epilogue &e, int m, int n, float
         return;
     }
     v = apply_act(v, e.act);
+    if (e.row_scale) v *= e.row_scale[(size_t)m * e.rs_ld + n / e.rs_cols];
     size_t i = (size_t)m * e.ldo + n;
-    if (e.out_half)
+    if (e.out_half == OUT_BF16)
+        static_cast<__nv_bfloat16 *>(e.out)[i] = __float2bfloat16_rn(v);
+    else if (e.out_half)
         static_cast<__half *>(e.out)[i] = __float2half_rn(v);
     else
         static_cast<float *>(e.out)[i] = v;
@@ -69,6 +86,23 @@ __device__ __forceinline__ void epi_store(const Epilogue &e, int m, int n, float
 // into e.pos_off by the caller (it is not dereferenced here for the vector path).
 __device__ __forceinline__ void epi_store4(const Epilogue &e, int m, int n, float4 v, int N) {
     if (e.no_store) return;
+    if (e.mode == EPI_GLU) { // N and ldo are multiples of 4
+        if (n >= N) return;
+        const size_t i = (size_t)m * e.ldo + (n >> 1);
+        *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(e.out) + i) =
+            pack_bf16x2(apply_act(v.x, e.act) * v.z, apply_act(v.y, e.act) * v.w);
+        return;
+    }
+    if (e.mode == EPI_ROPE) {
+        if (n >= N) return;
+        const int p = (n % e.rope_head - e.rope_at) >> 1;
+        if (p >= 0 && p < e.rope_pairs) {
+            const float2 *t = e.rope_tab + (size_t)row_pos(e.rows, m) * e.rope_pairs + p;
+            const float2 c0 = t[0];
+            const float2 c1 = p + 1 < e.rope_pairs ? t[1] : make_float2(1.0f, 0.0f);
+            v = make_float4(v.x * c0.x - v.y * c0.y, v.y * c0.x + v.x * c0.y, v.z * c1.x - v.w * c1.y, v.w * c1.x + v.z * c1.y);
+        }
+    }
     const bool vec = (n + 3 < N) && ((e.ldo & 3) == 0) && (e.pos_ptr == nullptr);
     if (!vec) {
         if (n < N) epi_store(e, m, n, v.x);
@@ -103,11 +137,13 @@ __device__ __forceinline__ void epi_store4(const Epilogue &e, int m, int n, floa
     }
     v.x = apply_act(v.x, e.act); v.y = apply_act(v.y, e.act);
     v.z = apply_act(v.z, e.act); v.w = apply_act(v.w, e.act);
+    if (e.row_scale) {
+        const float rs = e.row_scale[(size_t)m * e.rs_ld + n / e.rs_cols];
+        v.x *= rs; v.y *= rs; v.z *= rs; v.w *= rs;
+    }
     const size_t i = (size_t)m * e.ldo + n;
     if (e.out_half) {
-        __half2 lo = __floats2half2_rn(v.x, v.y), hi = __floats2half2_rn(v.z, v.w);
-        *reinterpret_cast<uint2 *>(static_cast<__half *>(e.out) + i) =
-            make_uint2(*reinterpret_cast<uint32_t *>(&lo), *reinterpret_cast<uint32_t *>(&hi));
+        *reinterpret_cast<uint2 *>(static_cast<__half *>(e.out) + i) = make_uint2(epi_pack2(e, v.x, v.y), epi_pack2(e, v.z, v.w));
     } else {
         *reinterpret_cast<float4 *>(static_cast<float *>(e.out) + i) = v;
     }
@@ -304,6 +340,11 @@ template <>
 __device__ __forceinline__ float load_as_float<float>(const float *p, size_t i) { return p[i]; }
 template <>
 __device__ __forceinline__ float load_as_float<__half>(const __half *p, size_t i) { return __half2float(p[i]); }
+template <>
+__device__ __forceinline__ float load_as_float<__nv_bfloat16>(const __nv_bfloat16 *p, size_t i) { return __bfloat162float(p[i]); }
+__device__ __forceinline__ void store_from_float(float *p, float v) { *p = v; }
+__device__ __forceinline__ void store_from_float(__half *p, float v) { *p = __float2half_rn(v); }
+__device__ __forceinline__ void store_from_float(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
 
 // Unpacks one 32-bit word of the tiled int4 layout (nibble positions 0..7 = k offsets
 // 0,2,4,6,1,3,5,7, each stored +8) into four half2 holding the exact integers (k0,k1) (k2,k3)

@@ -213,24 +213,29 @@ int embed_one(b200nn_gpt2 *m, Workspace &ws, const uint32_t *ids_host, int S, in
 }
 
 // Prefill of one prompt through all layers; logits of the last position end up in ws1.logits.
-int prefill_one(b200nn_gpt2 *m, b200nn_kvcache &kv, Workspace &ws1, const uint32_t *prompt, int n) {
+int prefill_one(b200nn_lm *m, b200nn_kvcache &kv, Workspace &ws1, const uint32_t *prompt, int n) {
     b200nn_ctx *ctx = m->ctx;
+    for (int i = 0; i < n; ++i)
+        if (prompt[i] >= (uint32_t)m->vocab()) return set_error(ctx, B200NN_ERR_DIM, "token id out of range for vocab_size");
+    const int part = kv.portion ? std::min<int>(n, (int)kv.portion) : n;
     Workspace wsp;
-    TRY(workspace_alloc(m, (size_t)n, 1, &wsp));
-    const bool ah = model_act_half(m, n);
-    TRY(embed_one(m, wsp, prompt, n, 0));
-    TRY(run_blocks(m, wsp, kv, 1, n, nullptr, 0, ah, nullptr));
+    TRY(m->workspace_init((size_t)part, 1, &wsp));
+    for (int p0 = 0; p0 < n; p0 += part) {
+        const int k = std::min(part, n - p0);
+        TRY(m->pass_prompt(wsp, kv, {PassEntry{0, p0, k}}, prompt + p0));
+        if (p0 + k == n)
+            TRY(launch_gather_last_rows(ctx, (const float *)wsp.x->p, 1, k, m->width(), (float *)ws1.last_x->p));
+    }
     kv.len = (size_t)n;
-    TRY(launch_gather_last_rows(ctx, (const float *)wsp.x->p, 1, n, m->cfg.n_embd, (float *)ws1.last_x->p));
-    TRY(run_head(m, ws1, (const float *)ws1.last_x->p, 1, model_act_half(m, 1), nullptr));
+    TRY(m->head(ws1, (const float *)ws1.last_x->p, 1, nullptr));
     CK(ctx, cudaStreamSynchronize(ctx->stream)); // wsp goes out of scope
     return B200NN_OK;
 }
 
 // The k best of ws.logits row 0 (scaled by 1/temp) -> host, then the reference's draw.
-int sample_row(b200nn_gpt2 *m, Workspace &ws, size_t k, float temp, uint64_t *rng, uint32_t *token) {
+int sample_row(b200nn_lm *m, Workspace &ws, size_t k, float temp, uint64_t *rng, uint32_t *token) {
     b200nn_ctx *ctx = m->ctx;
-    const int V = m->cfg.vocab_size;
+    const int V = m->vocab();
     const size_t kk = std::min<size_t>(k, (size_t)V);
     TRY(ensure_scratch(ctx, (size_t)V * 4 + kk * 8 + 64, 0));
     float *scaled = ctx->scratch;
@@ -272,10 +277,15 @@ int argmax_row(b200nn_gpt2 *m, Workspace &ws, uint32_t *token) {
 extern "C" int32_t b200nn_gpt2_generate_cached_sampling(b200nn_gpt2 *m, const uint32_t *prompt, size_t prompt_len,
                                                         size_t max_new, size_t top_k, float temperature,
                                                         uint64_t *rng_state, uint32_t *out_tokens, size_t *n_out) {
+    return b200nn_lm_generate_sampling(m, prompt, prompt_len, max_new, top_k, temperature, rng_state, out_tokens, n_out);
+}
+extern "C" int32_t b200nn_lm_generate_sampling(b200nn_lm *m, const uint32_t *prompt, size_t prompt_len, size_t max_new,
+                                               size_t top_k, float temperature, uint64_t *rng_state, uint32_t *out_tokens,
+                                               size_t *n_out) {
     if (!m || !prompt || !rng_state || !out_tokens || !n_out) return B200NN_ERR_ARG;
     b200nn_ctx *ctx = m->ctx;
     if (prompt_len == 0 || top_k == 0) return set_error(ctx, B200NN_ERR_SHAPE, "sampling: empty prompt or top_k == 0");
-    if (prompt_len + max_new > (size_t)m->cfg.n_positions)
+    if (m->max_positions() && prompt_len + max_new > m->max_positions())
         return set_error(ctx, B200NN_ERR_DIM, "sampling: prompt_len + max_new exceeds n_positions");
     CK(ctx, cudaSetDevice(ctx->device));
     const float temp = clamp_temperature(temperature);
@@ -284,21 +294,20 @@ extern "C" int32_t b200nn_gpt2_generate_cached_sampling(b200nn_gpt2 *m, const ui
     *n_out = n;
     if (max_new == 0) return B200NN_OK;
     CacheGuard g;
-    TRY(b200nn_kvcache_create(m, 1, prompt_len + max_new, &g.c));
+    TRY(b200nn_lm_cache_create(m, 1, prompt_len + max_new, &g.c));
     b200nn_kvcache &kv = *g.c;
     Workspace ws;
-    TRY(workspace_alloc(m, 1, 1, &ws));
+    TRY(m->workspace_init(1, 1, &ws));
     TRY(prefill_one(m, kv, ws, prompt, (int)prompt_len));
     uint32_t tok = 0;
     TRY(sample_row(m, ws, top_k, temp, rng_state, &tok));
     for (size_t step = 0;; ++step) {
-        if (tok == 50256u) break; // stop before appending (gpt2.rs:958-960, 970-972)
+        if (m->eos() >= 0 && tok == (uint32_t)m->eos()) break; // stop before appending (gpt2.rs:958-960, 970-972)
         out_tokens[n++] = tok;
         if (step + 1 >= max_new) break;
-        TRY(embed_one(m, ws, &tok, 1, (int)kv.len));
-        TRY(run_blocks(m, ws, kv, 1, 1, nullptr, (int)kv.len, model_act_half(m, 1), nullptr));
+        TRY(m->pass_prompt(ws, kv, {PassEntry{0, (int)kv.len, 1}}, &tok));
         kv.len += 1;
-        TRY(run_head(m, ws, (const float *)ws.x->p, 1, model_act_half(m, 1), nullptr));
+        TRY(m->head(ws, (const float *)ws.x->p, 1, nullptr));
         TRY(sample_row(m, ws, top_k, temp, rng_state, &tok));
     }
     *n_out = n;

@@ -45,6 +45,28 @@ enum : uint32_t { ERR_EMPTY = 0x201, ERR_FULL, ERR_ACC };
 constexpr int BK = 64;                 // fp16 elements per K block = one 128-byte swizzle row
 constexpr int W_BYTES = 128 * BK * 2;  // weight box: 128 features x 64 k
 
+// What the operands are besides plain fp16 matrices.  idesc_bits: operand-format bits of the instruction
+// descriptor (0: fp16, tc::UMMA_BF16: bfloat16; always the same for both operands).  A block-diagonal Linear
+// (groups > 1) has group_tiles feature tiles per group: tile nt multiplies the activation columns from
+// (nt / group_tiles) * group_kx on and its group_n features start at output column
+// (nt / group_tiles) * group_stride.
+struct OperandForm {
+    uint32_t idesc_bits = 0;
+    int group_tiles = 0x7fffffff, group_kx = 0, group_n = 0x7fffffff, group_stride = 0;
+};
+// Output column of a tile's feature (column n of the padded weight); lim: the number of columns from which on
+// nothing may be stored (N, or the end of the feature's group; 0 for a padding feature of a group).
+__device__ __forceinline__ int out_column(const OperandForm &f, int nt, int n, int N, int *lim) {
+    const int g = nt / f.group_tiles;
+    if (f.group_stride == 0) {
+        *lim = N;
+        return n;
+    }
+    const int local = n - g * f.group_tiles * 128;
+    *lim = local < f.group_n ? g * f.group_stride + f.group_n : 0;
+    return g * f.group_stride + local;
+}
+
 template <int NTHREADS>
 __device__ __forceinline__ void bar_sync_epi() {
     asm volatile("bar.sync 1, %0;" ::"n"(NTHREADS) : "memory");
@@ -56,7 +78,7 @@ template <int MB, int NS, int NE, int TW>
 __global__ void __launch_bounds__(64 + 128 * NE, 1)
 f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_w2,
                    const __grid_constant__ CUtensorMap tmap_x, int M, int N, int k_blocks, int kb_per_split,
-                   int cluster_mode, Epilogue epi, uint32_t *__restrict__ dev_err) {
+                   int cluster_mode, OperandForm form, Epilogue epi, uint32_t *__restrict__ dev_err) {
     constexpr int X_BYTES = MB * BK * 2;
     constexpr int WT_BYTES = TW * W_BYTES; // the weight boxes of one stage, hi then lo
     constexpr int STAGE = WT_BYTES + X_BYTES;
@@ -98,7 +120,9 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
     const uint32_t tmem_base = *reinterpret_cast<volatile uint32_t *>(gen_base + (tmem_slot - base));
     // the epilogue's per-thread constants (filled by the epilogue warps, used in both of its places):
     // lane l owns features 4l..4l+3 of a token row
-    const int n4 = nt * 128 + lane * 4;
+    int n_lim;
+    const int n4 = out_column(form, nt, nt * 128 + lane * 4, N, &n_lim);
+    const int kx = (nt / form.group_tiles) * form.group_kx; // first activation column
     float4 b4 = make_float4(0.f, 0.f, 0.f, 0.f);
     Epilogue e2 = epi; // the device-side position is read once per thread
     e2.pos_ptr = nullptr;
@@ -118,7 +142,7 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         pdl_wait();
         if (tc::elect_one()) {
             for (int i = 0; i < npre; ++i)
-                tc::tma_load_2d(base + i * STAGE + WT_BYTES, &tmap_x, (kb0 + i) * BK, mt * MB, full + 8 * i);
+                tc::tma_load_2d(base + i * STAGE + WT_BYTES, &tmap_x, kx + (kb0 + i) * BK, mt * MB, full + 8 * i);
         }
         __syncwarp();
         int s = 0;
@@ -129,14 +153,14 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
                 tc::mbar_expect_tx(full + 8 * s, STAGE);
                 tc::tma_load_2d(base + s * STAGE, &tmap_w, (kb0 + i) * BK, nt * 128, full + 8 * s);
                 if (TW == 2) tc::tma_load_2d(base + s * STAGE + W_BYTES, &tmap_w2, (kb0 + i) * BK, nt * 128, full + 8 * s);
-                tc::tma_load_2d(base + s * STAGE + WT_BYTES, &tmap_x, (kb0 + i) * BK, mt * MB, full + 8 * s);
+                tc::tma_load_2d(base + s * STAGE + WT_BYTES, &tmap_x, kx + (kb0 + i) * BK, mt * MB, full + 8 * s);
             }
             __syncwarp();
             if (++s == NS) { s = 0; ph ^= 1; }
         }
     } else if (warp == 1) {
         // ---- MMA issue: the whole warp runs the loop, one elected lane issues ----
-        constexpr uint32_t idesc = tc::umma_idesc_f16(128, MB);
+        const uint32_t idesc = tc::umma_idesc_f16(128, MB) | form.idesc_bits;
         const uint64_t d0 = tc::umma_desc_sw128(base);
         bool ok = true;
         int s = 0;
@@ -174,7 +198,7 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         const int colh = w8 >> 2;         // the NE warps of a quadrant split the token columns
         pdl_wait(); // the epilogue touches buffers the previous kernel may still be using
         // bias and the device-side position are fetched under the wait for the accumulator
-        b4 = epi_bias4(epi, n4, N);
+        b4 = epi_bias4(epi, n4, n_lim);
         if (epi.mode == EPI_QKV && epi.pos_ptr) e2.pos_off = epi.pos_off + *epi.pos_ptr;
         // (the vote keeps the warp converged for the warp-collective wait)
         if (!__any_sync(0xffffffffu, abort_flag != 0)) tc::mbar_wait(acc_full, 0, &abort_flag, dev_err, ERR_ACC);
@@ -205,8 +229,8 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
             if (splits == 1) {
                 for (int c = w8; c < rows; c += NW) {
                     const float4 v = f4_add(stage4[c * 32 + lane], b4);
-                    epi_store4(e2, mt * MB + c, n4, v, N);
-                    if (epi.amax_val) epi_argmax4(epi, mt * MB + c, n4, v, N);
+                    epi_store4(e2, mt * MB + c, n4, v, n_lim);
+                    if (epi.amax_val) epi_argmax4(epi, mt * MB + c, n4, v, n_lim);
                 }
             } else if (epi.mode == EPI_RESID) {
                 // every split adds its partial tile into the f32 residual stream with vector
@@ -214,7 +238,7 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
                 // fixed, so the last bits of the sum can differ between runs.
                 const float4 add0 = (split == 0) ? b4 : make_float4(0.f, 0.f, 0.f, 0.f);
                 for (int c = w8; c < rows; c += NW)
-                    epi_resid_red4(epi, mt * MB + c, n4, f4_add(stage4[c * 32 + lane], add0), N);
+                    epi_resid_red4(epi, mt * MB + c, n4, f4_add(stage4[c * 32 + lane], add0), n_lim);
             } // else: the splits are one cluster, summed below
         }
     }
@@ -234,8 +258,8 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
                 float4 sum = b4;
                 for (int sp = 0; sp < splits; ++sp)
                     sum = f4_add(sum, cluster.map_shared_rank(stage4, sp)[c * 32 + lane]);
-                epi_store4(e2, mt * MB + c, n4, sum, N);
-                if (epi.amax_val) epi_argmax4(epi, mt * MB + c, n4, sum, N);
+                epi_store4(e2, mt * MB + c, n4, sum, n_lim);
+                if (epi.amax_val) epi_argmax4(epi, mt * MB + c, n4, sum, n_lim);
             }
         }
         cluster.sync(); // no block leaves while its shared memory may still be read
@@ -278,7 +302,7 @@ template <int MB, int NS, int NE, int TW>
 __global__ void __launch_bounds__(64 + 128 * NE, 1)
 f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_w2,
                               const __grid_constant__ CUtensorMap tmap_x, int M, int N, int k_blocks, int n_tiles,
-                              int total_tiles, Epilogue epi, uint32_t *__restrict__ dev_err) {
+                              int total_tiles, OperandForm form, Epilogue epi, uint32_t *__restrict__ dev_err) {
     constexpr int X_BYTES = MB * BK * 2;
     constexpr int WT_BYTES = TW * W_BYTES;
     constexpr int STAGE = WT_BYTES + X_BYTES;
@@ -332,6 +356,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
         bool ok = true;
         for (int t = blockIdx.x; ok && t < total_tiles; t += gridDim.x) {
             const int mt = t / n_tiles, nt = t - mt * n_tiles;
+            const int kx = (nt / form.group_tiles) * form.group_kx;
             for (int kb = 0; kb < k_blocks; ++kb) {
                 ok = tc::mbar_wait(empty + 8 * s, ph, &abort_flag, dev_err, ERR_EMPTY);
                 if (!ok) break;
@@ -339,7 +364,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
                     tc::mbar_expect_tx(full + 8 * s, STAGE);
                     tc::tma_load_2d(base + s * STAGE, &tmap_w, kb * BK, nt * 128, full + 8 * s);
                     if (TW == 2) tc::tma_load_2d(base + s * STAGE + W_BYTES, &tmap_w2, kb * BK, nt * 128, full + 8 * s);
-                    tc::tma_load_2d(base + s * STAGE + WT_BYTES, &tmap_x, kb * BK, mt * MB, full + 8 * s);
+                    tc::tma_load_2d(base + s * STAGE + WT_BYTES, &tmap_x, kx + kb * BK, mt * MB, full + 8 * s);
                 }
                 __syncwarp();
                 if (++s == NS) { s = 0; ph ^= 1; }
@@ -347,7 +372,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
         }
     } else if (warp == 1) {
         // ---- MMA issue ----
-        constexpr uint32_t idesc = tc::umma_idesc_f16(128, MB);
+        const uint32_t idesc = tc::umma_idesc_f16(128, MB) | form.idesc_bits;
         const uint64_t d0 = tc::umma_desc_sw128(base);
         int s = 0;
         uint32_t ph = 0;
@@ -402,8 +427,9 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
         for (int t = blockIdx.x; t < total_tiles; t += gridDim.x, ++j) {
             const int b = j & 1;
             const int mt = t / n_tiles, nt = t - mt * n_tiles;
-            const int n4 = nt * 128 + lane * 4;
-            const float4 b4 = epi_bias4(epi, n4, N); // fetched under the wait for the accumulator
+            int n_lim;
+            const int n4 = out_column(form, nt, nt * 128 + lane * 4, N, &n_lim);
+            const float4 b4 = epi_bias4(epi, n4, n_lim); // fetched under the wait for the accumulator
             bool ok = true;
             if (!__any_sync(0xffffffffu, abort_flag != 0))
                 ok = tc::mbar_wait(acc_full + 8 * b, (j >> 1) & 1, &abort_flag, dev_err, ERR_ACC);
@@ -428,12 +454,12 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
                     // this block is the only one that adds to these elements: a reduction at L2 does
                     // the read-modify-write there, with no load for the warp to wait on
                     for (int c = w8; c < lim; c += NW)
-                        epi_resid_red4(epi, mt * MB + c0 + c, n4, f4_add(stage4[c * 32 + lane], b4), N);
+                        epi_resid_red4(epi, mt * MB + c0 + c, n4, f4_add(stage4[c * 32 + lane], b4), n_lim);
                 } else {
                     for (int c = w8; c < lim; c += NW) {
                         const float4 v = f4_add(stage4[c * 32 + lane], b4);
-                        epi_store4(e2, mt * MB + c0 + c, n4, v, N);
-                        if (epi.amax_val) epi_argmax4(epi, mt * MB + c0 + c, n4, v, N);
+                        epi_store4(e2, mt * MB + c0 + c, n4, v, n_lim);
+                        if (epi.amax_val) epi_argmax4(epi, mt * MB + c0 + c, n4, v, n_lim);
                     }
                 }
                 bar_sync_epi<EPI>(); // the stage is free for the next pass
@@ -458,13 +484,14 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t
                                   const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
                                   CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-// fp16 matrix [rows, K] row-major as a 2-D tensor map with a [box_rows x 64] box and 128-byte swizzle
-int make_map(b200nn_ctx *ctx, const void *p, int rows, int K, int box_rows, CUtensorMap *out) {
+// 16-bit matrix [rows, K] with rows ld elements apart as a 2-D tensor map with a [box_rows x 64] box and
+// 128-byte swizzle
+int make_map(b200nn_ctx *ctx, const void *p, int rows, int K, int ld, int box_rows, bool bf16, CUtensorMap *out) {
     cuuint64_t gdim[2] = {(cuuint64_t)K, (cuuint64_t)rows};
-    cuuint64_t gstride[1] = {(cuuint64_t)K * sizeof(__half)};
+    cuuint64_t gstride[1] = {(cuuint64_t)ld * sizeof(__half)};
     cuuint32_t box[2] = {BK, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
-    CUresult r = ((EncodeTiledFn)ctx->encode_tiled)(out, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void *)p, gdim, gstride, box, estr,
+    CUresult r = ((EncodeTiledFn)ctx->encode_tiled)(out, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, (void *)p, gdim, gstride, box, estr,
                                                     CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
                                                     CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) return set_error(ctx, B200NN_ERR_CUDA, "cuTensorMapEncodeTiled failed: " + std::to_string((int)r));
@@ -479,6 +506,9 @@ struct WOperand {
     const __half *hi, *lo;
     int N, K;
     bool constant;
+    int ldx = 0, kx_total = 0; // row stride of the activations and the columns they have (0: K)
+    OperandForm form{};
+    bool bf16() const { return form.idesc_bits != 0; }
 };
 
 template <int MB, int NS, int NE, int TW>
@@ -495,9 +525,9 @@ int launch_cfg(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M, const
         attr_done[ctx->device & 15] = true;
     }
     CUtensorMap tmap_w, tmap_w2, tmap_x;
-    TRY(make_map(ctx, w.hi, w.N, w.K, 128, &tmap_w));
-    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, 128, &tmap_w2));
-    TRY(make_map(ctx, x, M, w.K, MB, &tmap_x));
+    TRY(make_map(ctx, w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w));
+    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w2));
+    TRY(make_map(ctx, x, M, w.kx_total ? w.kx_total : w.K, w.ldx ? w.ldx : w.K, MB, w.bf16(), &tmap_x));
 
     const int k_blocks = (w.K + BK - 1) / BK;
     const int n_tiles = (w.N + 127) / 128, m_tiles = (M + MB - 1) / MB;
@@ -538,7 +568,7 @@ int launch_cfg(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M, const
     }
     cfg.attrs = attr;
     cfg.numAttrs = na;
-    CK(ctx, cudaLaunchKernelEx(&cfg, kern, tmap_w, tmap_w2, tmap_x, M, w.N, k_blocks, per, cluster_mode, epi, ctx->dev_err));
+    CK(ctx, cudaLaunchKernelEx(&cfg, kern, tmap_w, tmap_w2, tmap_x, M, w.N, k_blocks, per, cluster_mode, w.form, epi, ctx->dev_err));
     CK_LAUNCH(ctx, "f16_gemm_tc_kernel");
     return B200NN_OK;
 }
@@ -558,9 +588,9 @@ int launch_persistent(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M
         attr_done[ctx->device & 15] = true;
     }
     CUtensorMap tmap_w, tmap_w2, tmap_x;
-    TRY(make_map(ctx, w.hi, w.N, w.K, 128, &tmap_w));
-    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, 128, &tmap_w2));
-    TRY(make_map(ctx, x, M, w.K, MB, &tmap_x));
+    TRY(make_map(ctx, w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w));
+    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w2));
+    TRY(make_map(ctx, x, M, w.kx_total ? w.kx_total : w.K, w.ldx ? w.ldx : w.K, MB, w.bf16(), &tmap_x));
     const int k_blocks = (w.K + BK - 1) / BK;
     const int n_tiles = (w.N + 127) / 128, m_tiles = (M + MB - 1) / MB;
     const int total = n_tiles * m_tiles;
@@ -574,7 +604,7 @@ int launch_persistent(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = (ctx->pdl && w.constant) ? 1 : 0;
-    CK(ctx, cudaLaunchKernelEx(&cfg, kern, tmap_w, tmap_w2, tmap_x, M, w.N, k_blocks, n_tiles, total, epi, ctx->dev_err));
+    CK(ctx, cudaLaunchKernelEx(&cfg, kern, tmap_w, tmap_w2, tmap_x, M, w.N, k_blocks, n_tiles, total, w.form, epi, ctx->dev_err));
     CK_LAUNCH(ctx, "f16_gemm_tc_persistent_kernel");
     return B200NN_OK;
 }
@@ -661,7 +691,7 @@ int4_dequant_f16_kernel(const uint8_t *__restrict__ tiles, const __half *__restr
 
 // The tensor maps need 16-byte aligned bases and row strides: K a multiple of 8.
 bool f16_gemm_tc_supported(const b200nn_ctx *ctx, const F32Weight &w, int M) {
-    return ctx->f32_tc && ctx->encode_tiled && w.w_nk_h && M > 4 && (w.K % 8) == 0;
+    return ctx->f32_tc && !w.exact && ctx->encode_tiled && w.w_nk_h && M > 4 && (w.K % 8) == 0;
 }
 
 int launch_f16_gemm_tc(b200nn_ctx *ctx, const F32Weight &w, const __half *x, int M, const Epilogue &epi) {
@@ -670,6 +700,24 @@ int launch_f16_gemm_tc(b200nn_ctx *ctx, const F32Weight &w, const __half *x, int
     const __half *hi = (const __half *)w.w_nk_h->p;
     const WOperand op{hi, hi + (size_t)w.N * w.K, w.N, w.K, true};
     return launch_terms(ctx, op, ctx->f32_tc == 1 ? 1 : 2, x, M, epi);
+}
+
+// bfloat16 weight and activations, any row count.
+int launch_b16_linear(b200nn_ctx *ctx, const B16Weight &w, const __nv_bfloat16 *x, int ldx, int M, const Epilogue &epi) {
+    if (M <= 0) return B200NN_OK;
+    if (!ctx->encode_tiled) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "cuTensorMapEncodeTiled is unavailable");
+    if (((uintptr_t)x & 15) || (ldx & 7)) return set_error(ctx, B200NN_ERR_ARG, "bf16 Linear: activations must be 16-byte aligned, rows a multiple of 8");
+    WOperand op{(const __half *)w.w_nk->p, nullptr, w.N, w.K, true};
+    op.ldx = ldx;
+    op.kx_total = w.K + (w.groups - 1) * w.group_kx;
+    op.form.idesc_bits = tc::UMMA_BF16;
+    if (w.groups > 1) {
+        op.form.group_tiles = w.group_tiles;
+        op.form.group_kx = w.group_kx;
+        op.form.group_n = w.group_n;
+        op.form.group_stride = w.group_stride;
+    }
+    return launch_terms(ctx, op, 1, (const __half *)x, M, epi);
 }
 
 // int4 Linear over the rows of a prefill pass: the weight is first written out as the [N,K] fp16

@@ -1,6 +1,7 @@
 // Small fused kernels of the GPT-2 path: LayerNorm (+residual), embedding gather, activations,
 // bias / residual adds, head split / concat, dtype conversion, greedy argmax.
 #include "device_utils.cuh"
+#include "hybrid.h"
 
 // ---------------------------------------------------------------------------------------------
 // LayerNorm: gamma*(x-mean)/sqrt(var+eps)+beta, biased variance (cpu_ref.rs:27-54).  One block per
@@ -553,5 +554,177 @@ int launch_tensor_transpose(b200nn_ctx *ctx, const float *in, float *out, const 
     if (n == 0) return B200NN_OK;
     tensor_transpose_kernel<<<(unsigned)((n + 255) / 256), 256, 0, ctx->stream>>>(in, out, n, td);
     CK_LAUNCH(ctx, "tensor_transpose_kernel");
+    return B200NN_OK;
+}
+
+// ---------------------------------------------------------------------------------------------
+// Pieces of the hybrid decoder: RMS norm, embedding without positions, gated products, row gather and the
+// block-diagonal f32 Linear.
+// ---------------------------------------------------------------------------------------------
+// x / sqrt(mean(x^2) + eps) * w, one block per row; output rows ldo apart.
+template <int VPT, typename TOut>
+__global__ void __launch_bounds__(256) rmsnorm_kernel(const float *__restrict__ x, const float *__restrict__ w, float eps, int d, int ldo,
+                                                      TOut *__restrict__ out) {
+    __shared__ float red[32];
+    const int row = blockIdx.x, tid = threadIdx.x;
+    pdl_trigger();
+    float g[VPT]; // constant: fetched before the wait
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) g[i] = tid + i * 256 < d ? w[tid + i * 256] : 0.0f;
+    pdl_wait();
+    float v[VPT], s = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+        v[i] = tid + i * 256 < d ? x[(size_t)row * d + tid + i * 256] : 0.0f;
+        s = fmaf(v[i], v[i], s);
+    }
+    const float r = 1.0f / sqrtf(block_sum(s, red) / (float)d + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i)
+        if (tid + i * 256 < d) store_from_float(out + (size_t)row * ldo + tid + i * 256, v[i] * r * g[i]);
+}
+
+// Many rows (prompt passes): one warp per row, the row in registers (NV float4 per lane); d a multiple of 4.
+template <int NV>
+__global__ void __launch_bounds__(256) rmsnorm_rows_kernel(const float *__restrict__ x, const float *__restrict__ w, float eps, int rows,
+                                                           int d, int ldo, __nv_bfloat16 *__restrict__ out) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, d4 = d >> 2;
+    pdl_trigger();
+    pdl_wait();
+    for (int row = blockIdx.x * 8 + warp; row < rows; row += gridDim.x * 8) {
+        const float4 *xr = reinterpret_cast<const float4 *>(x + (size_t)row * d);
+        float4 v[NV];
+        float s = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            v[i] = c < d4 ? __ldcs(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            s += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+        }
+        const float r = 1.0f / sqrtf(warp_sum(s) / (float)d + eps);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = lane + 32 * i;
+            if (c < d4) {
+                const float4 g = __ldg(reinterpret_cast<const float4 *>(w) + c);
+                reinterpret_cast<uint2 *>(out + (size_t)row * ldo)[c] =
+                    make_uint2(pack_bf16x2(v[i].x * r * g.x, v[i].y * r * g.y), pack_bf16x2(v[i].z * r * g.z, v[i].w * r * g.w));
+            }
+        }
+    }
+}
+
+int launch_rmsnorm(b200nn_ctx *ctx, const float *x, const float *w, float eps, int rows, int d, int ldo, void *out, int out_type) {
+    if (rows <= 0) return B200NN_OK;
+    if (d > 256 * 32) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "rms_norm: d > 8192");
+    if (out_type == OUT_BF16 && rows >= ctx->ln_rows_min && d % 4 == 0 && ldo % 4 == 0 && d <= 4096) {
+        const dim3 grid(std::min((rows + 7) / 8, 8 * ctx->sm_count));
+        const int nv = (d / 4 + 31) / 32;
+#define RMS_ROWS(N)                                                                                                        \
+    do {                                                                                                                   \
+        PREFER_SMEM_ONCE(rmsnorm_rows_kernel<N>);                                                                          \
+        launch_pdl(ctx, rmsnorm_rows_kernel<N>, grid, dim3(256), 0, x, w, eps, rows, d, ldo, (__nv_bfloat16 *)out);        \
+    } while (0)
+        if (nv <= 4) RMS_ROWS(4);
+        else if (nv <= 8) RMS_ROWS(8);
+        else if (nv <= 16) RMS_ROWS(16);
+        else RMS_ROWS(32);
+#undef RMS_ROWS
+        CK_LAUNCH(ctx, "rmsnorm_rows_kernel");
+        return B200NN_OK;
+    }
+#define RMS(V)                                                                                                             \
+    do {                                                                                                                   \
+        PREFER_SMEM_ONCE((rmsnorm_kernel<V, __nv_bfloat16>));                                                              \
+        PREFER_SMEM_ONCE((rmsnorm_kernel<V, float>));                                                                      \
+        if (out_type == OUT_BF16)                                                                                          \
+            launch_pdl(ctx, rmsnorm_kernel<V, __nv_bfloat16>, dim3(rows), dim3(256), 0, x, w, eps, d, ldo, (__nv_bfloat16 *)out); \
+        else                                                                                                               \
+            launch_pdl(ctx, rmsnorm_kernel<V, float>, dim3(rows), dim3(256), 0, x, w, eps, d, ldo, (float *)out);          \
+    } while (0)
+    const int vpt = (d + 255) / 256;
+    if (vpt <= 4) RMS(4);
+    else if (vpt <= 8) RMS(8);
+    else if (vpt <= 16) RMS(16);
+    else RMS(32);
+#undef RMS
+    CK_LAUNCH(ctx, "rmsnorm_kernel");
+    return B200NN_OK;
+}
+
+template <typename T>
+__global__ void embedding_rows_kernel(const uint32_t *__restrict__ ids, const T *__restrict__ table, int ldt, int d, int vocab,
+                                      float *__restrict__ out) {
+    const int r = blockIdx.x;
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t tok = min(ids[r], (uint32_t)vocab - 1); // ids are validated on the host; never read out of range
+    for (int j = threadIdx.x; j < d; j += blockDim.x) out[(size_t)r * d + j] = load_as_float<T>(table, (size_t)tok * ldt + j);
+}
+int launch_embedding_rows(b200nn_ctx *ctx, const uint32_t *ids, const void *table, bool b16, int ldt, int n_rows, int d, int vocab,
+                          float *out) {
+    if (n_rows <= 0) return B200NN_OK;
+    PREFER_SMEM_ONCE(embedding_rows_kernel<__nv_bfloat16>);
+    PREFER_SMEM_ONCE(embedding_rows_kernel<float>);
+    if (b16) launch_pdl(ctx, embedding_rows_kernel<__nv_bfloat16>, dim3(n_rows), dim3(256), 0, ids, (const __nv_bfloat16 *)table, ldt, d, vocab, out);
+    else launch_pdl(ctx, embedding_rows_kernel<float>, dim3(n_rows), dim3(256), 0, ids, (const float *)table, ldt, d, vocab, out);
+    CK_LAUNCH(ctx, "embedding_rows_kernel");
+    return B200NN_OK;
+}
+
+__global__ void glu_kernel(const float4 *__restrict__ gu, size_t quads, int act, float2 *__restrict__ out) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= quads) return;
+    const float4 v = gu[i];
+    out[i] = make_float2(apply_act(v.x, act) * v.z, apply_act(v.y, act) * v.w);
+}
+int launch_glu(b200nn_ctx *ctx, const float *gu, int rows, int n2, int act, float *out) {
+    const size_t quads = (size_t)rows * n2 / 4;
+    if (!quads) return B200NN_OK;
+    PREFER_SMEM_ONCE(glu_kernel);
+    launch_pdl(ctx, glu_kernel, dim3((unsigned)((quads + 255) / 256)), dim3(256), 0, (const float4 *)gu, quads, act, (float2 *)out);
+    CK_LAUNCH(ctx, "glu_kernel");
+    return B200NN_OK;
+}
+
+__global__ void gather_rows_kernel(const float *__restrict__ src, const int *__restrict__ idx, int d, float *__restrict__ dst) {
+    pdl_trigger();
+    pdl_wait();
+    const float *s = src + (size_t)idx[blockIdx.x] * d;
+    for (int j = threadIdx.x; j < d; j += blockDim.x) dst[(size_t)blockIdx.x * d + j] = s[j];
+}
+int launch_gather_rows(b200nn_ctx *ctx, const float *src, const int *idx, int n_rows, int d, float *dst) {
+    if (n_rows <= 0) return B200NN_OK;
+    PREFER_SMEM_ONCE(gather_rows_kernel);
+    launch_pdl(ctx, gather_rows_kernel, dim3(n_rows), dim3(256), 0, src, idx, d, dst);
+    CK_LAUNCH(ctx, "gather_rows_kernel");
+    return B200NN_OK;
+}
+
+// One warp per output: the weight rows are contiguous along K.
+__global__ void __launch_bounds__(256) grouped_f32_kernel(const float *__restrict__ w, int groups, int Ng, int Kg, const float *__restrict__ x,
+                                                          int ldx, int x_stride, int M, Epilogue epi, int out_stride) {
+    pdl_trigger();
+    pdl_wait();
+    const size_t unit = (size_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31;
+    if (unit >= (size_t)M * groups * Ng) return;
+    const int gn = (int)(unit % ((size_t)groups * Ng)), m = (int)(unit / ((size_t)groups * Ng)), g = gn / Ng, n = gn - g * Ng;
+    const float *wr = w + (size_t)gn * Kg, *xr = x + (size_t)m * ldx + (size_t)g * x_stride;
+    float a = 0.0f;
+    for (int k = lane; k < Kg; k += 32) a = fmaf(wr[k], xr[k], a);
+    a = warp_sum(a);
+    if (lane == 0) epi_apply(epi, m, g * out_stride + n, a);
+}
+int launch_grouped_f32(b200nn_ctx *ctx, const float *w, int groups, int Ng, int Kg, const float *x, int ldx, int x_stride, int M,
+                       const Epilogue &epi, int out_stride) {
+    const size_t units = (size_t)M * groups * Ng;
+    if (!units) return B200NN_OK;
+    PREFER_SMEM_ONCE(grouped_f32_kernel);
+    launch_pdl(ctx, grouped_f32_kernel, dim3((unsigned)((units + 7) / 8)), dim3(256), 0, w, groups, Ng, Kg, x, ldx, x_stride, M, epi,
+               out_stride);
+    CK_LAUNCH(ctx, "grouped_f32_kernel");
     return B200NN_OK;
 }

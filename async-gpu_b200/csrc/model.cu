@@ -6,7 +6,11 @@
 
 #include "model.h"
 
-int linear_forward(b200nn_ctx *ctx, const LinearAny &l, const void *x, bool x_half, int M, Epilogue epi) {
+int linear_forward(b200nn_ctx *ctx, const LinearAny &l, const void *x, bool x_half, int M, Epilogue epi, int ldx) {
+    if (l.b16) {
+        if (!x_half) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "a bfloat16 Linear takes bfloat16 activations");
+        return launch_b16_linear(ctx, l.b, static_cast<const __nv_bfloat16 *>(x), ldx ? ldx : l.b.K, M, epi);
+    }
     if (!epi.ln_stats) epi.bias = l.bias(); // a folded LayerNorm brings its own combined bias
     if (l.int4) return launch_int4_linear(ctx, l.q, x, x_half, M, epi);
     return launch_f32_linear(ctx, l.f, x, x_half, M, epi);
@@ -184,15 +188,6 @@ bool model_act_half(const b200nn_gpt2 *m, int rows) {
     if (rows <= m->ctx->gemv_max_rows) return false;
     return int4_gemm_tc_supported(b.qkv.q, rows) && int4_gemm_tc_supported(b.proj.q, rows) &&
            int4_gemm_tc_supported(b.fc.q, rows) && int4_gemm_tc_supported(b.fcproj.q, rows);
-}
-
-static inline void prof_mark(b200nn_ctx *ctx, StepProfile *p, int fam) {
-    if (!p) return;
-    cudaEvent_t e;
-    cudaEventCreate(&e);
-    cudaEventRecord(e, ctx->stream);
-    p->ev.push_back(e);
-    p->fam.push_back(fam);
 }
 
 // The seven launches of one transformer block, each on its own so that the forward pass (all of them,
@@ -390,4 +385,80 @@ int run_head_pick(b200nn_gpt2 *m, Workspace &ws, const float *x, int rows, bool 
     TRY(linear_forward(ctx, m->lm_head, ws.last_ln->p, head_half, rows, e));
     prof_mark(ctx, prof, B200NN_PROF_LM_HEAD);
     return launch_argmax_entries(ctx, e.amax_val, e.amax_idx, rows, e.amax_entries, V, keep_last, tok_out);
+}
+
+// ---------------------------------------------------------------------------------------------
+// the family's side of b200nn_lm
+// ---------------------------------------------------------------------------------------------
+b200nn_kvcache::b200nn_kvcache() = default;
+b200nn_kvcache::~b200nn_kvcache() = default;
+
+int b200nn_gpt2::cache_init(size_t batch, size_t cap, b200nn_kvcache *c) {
+    if (cap > (size_t)cfg.n_positions) return set_error(ctx, B200NN_ERR_DIM, "KvCache: capacity exceeds n_positions");
+    c->n_head = (size_t)cfg.n_head;
+    const size_t bytes = (size_t)cfg.n_layer * batch * cfg.n_embd * cap * sizeof(__half);
+    TRY(dev_alloc(ctx, bytes, &c->k));
+    return dev_alloc(ctx, bytes, &c->v);
+}
+
+int b200nn_gpt2::workspace_init(size_t rows, size_t logit_rows, Workspace *ws) { return workspace_alloc(this, rows, logit_rows, ws); }
+
+// Entries that are neighbouring slots of equal past and length run as one batch through a view of the cache
+// that starts at the first of them.
+int b200nn_gpt2::pass_prompt(Workspace &ws, b200nn_kvcache &kv, const std::vector<PassEntry> &entries, const uint32_t *ids_host) {
+    size_t row = 0;
+    Workspace sub = ws; // shares the buffers; x and ids move along with the rows
+    for (size_t i = 0; i < entries.size();) {
+        size_t j = i + 1;
+        while (j < entries.size() && entries[j].slot == entries[j - 1].slot + 1 && entries[j].past == entries[i].past &&
+               entries[j].n == entries[i].n)
+            ++j;
+        const int B = (int)(j - i), S = entries[i].n, past = entries[i].past, T = B * S;
+        if (row + T > ws.rows) return set_error(ctx, B200NN_ERR_SHAPE, "workspace too small");
+        if ((size_t)past + S > kv.cap) return set_error(ctx, B200NN_ERR_DIM, "KV cache capacity exceeded");
+        auto borrowed = [](void *p) { // an address inside another buffer: nothing to free
+            return std::shared_ptr<DevBuf>(new DevBuf{p}, [](DevBuf *b) {
+                b->p = nullptr;
+                delete b;
+            });
+        };
+        b200nn_kvcache view;
+        view.m = this;
+        view.batch = kv.batch; // layer stride of the full cache
+        view.cap = kv.cap;
+        view.n_head = kv.n_head;
+        const size_t seq_off = (size_t)entries[i].slot * cfg.n_head * kv.cap * 64;
+        view.k = borrowed((__half *)kv.k->p + seq_off);
+        view.v = borrowed((__half *)kv.v->p + seq_off);
+        sub.x = borrowed((float *)ws.x->p + row * cfg.n_embd);
+        CK(ctx, cudaMemcpyAsync(ws.ids->p, ids_host + row, (size_t)T * 4, cudaMemcpyHostToDevice, ctx->stream));
+        TRY(launch_embedding(ctx, (const uint32_t *)ws.ids->p, (const float *)wte->p, (const float *)wpe->p, T, cfg.n_embd, S,
+                             nullptr, past, cfg.vocab_size, cfg.n_positions, (float *)sub.x->p));
+        TRY(run_blocks(this, sub, view, B, S, nullptr, past, model_act_half(this, T), nullptr));
+        row += T;
+        i = j;
+    }
+    return B200NN_OK;
+}
+
+int b200nn_gpt2::pass_decode(Workspace &ws, b200nn_kvcache &kv, const int *pos_ptr, StepProfile *prof) {
+    const int B = (int)kv.batch, d = cfg.n_embd;
+    const bool fold = ws.ln_stats && ctx->ln_fold && model_ln_fold_supported(this, B);
+    if (fold)
+        TRY(launch_embedding_ln(ctx, (const uint32_t *)ws.tok->p, (const float *)wte->p, (const float *)wpe->p, B, d, pos_ptr,
+                                cfg.vocab_size, cfg.n_positions, (float *)ws.x->p, (const float *)blocks[0].ln1_g->p,
+                                (__half *)ws.ln->p, ws.ln_slot(0), ws.ln_nt));
+    else
+        TRY(launch_embedding(ctx, (const uint32_t *)ws.tok->p, (const float *)wte->p, (const float *)wpe->p, B, d, 1, pos_ptr, 0,
+                             cfg.vocab_size, cfg.n_positions, (float *)ws.x->p));
+    prof_mark(ctx, prof, B200NN_PROF_EMBED);
+    return run_blocks(this, ws, kv, B, 1, pos_ptr, 0, model_act_half(this, B), prof, fold);
+}
+
+int b200nn_gpt2::head(Workspace &ws, const float *x, int rows, StepProfile *prof) {
+    return run_head(this, ws, x, rows, model_act_half(this, rows), prof);
+}
+int b200nn_gpt2::head_pick(Workspace &ws, const float *x, int rows, bool keep_last, bool tokens_only, uint32_t *tok_out,
+                           StepProfile *prof) {
+    return run_head_pick(this, ws, x, rows, model_act_half(this, rows), keep_last, tokens_only, tok_out, prof);
 }

@@ -3,9 +3,10 @@
 #include "common.h"
 
 struct LinearAny {
-    bool int4 = false;
+    bool int4 = false, b16 = false;
     Int4Weight q;
     F32Weight f;
+    B16Weight b;
     int K = 0, N = 0;
     const float *bias() const {
         const std::shared_ptr<DevBuf> &b = int4 ? q.bias : f.bias;
@@ -13,11 +14,14 @@ struct LinearAny {
     }
     // algorithmic bytes of the weight side (nibbles + fp16 scales, or f32 weights) plus bias
     size_t weight_bytes() const {
+        if (b16) return (size_t)K * N * 2;
         if (int4) return (size_t)K * N / 2 + (size_t)q.n_groups * N * 2 + (q.bias ? (size_t)N * 4 : 0);
         return (size_t)K * N * 4 + (f.bias ? (size_t)N * 4 : 0);
     }
 };
-int linear_forward(b200nn_ctx *ctx, const LinearAny &l, const void *x, bool x_half, int M, Epilogue epi);
+// x_half: the activations are 16-bit (fp16, or bfloat16 for a bfloat16 weight), K elements per row unless
+// ldx says otherwise (bfloat16 only).
+int linear_forward(b200nn_ctx *ctx, const LinearAny &l, const void *x, bool x_half, int M, Epilogue epi, int ldx = 0);
 
 struct b200nn_linear {
     b200nn_ctx *ctx;
@@ -53,8 +57,52 @@ struct BlockW {
     std::shared_ptr<DevBuf> qkv_gsum, qkv_bc, fc_gsum, fc_bc;
 };
 
-struct b200nn_gpt2 {
+struct Workspace;
+struct StepProfile;
+
+// `n` new tokens of the sequence in cache slot `slot`, at positions past .. past + n - 1.
+struct PassEntry {
+    int slot, past, n;
+};
+
+// A decoder-only language model as the cache, the decode session, the serving step and the generate loops see
+// it: the model families derive from it.  A pass embeds token rows, runs every layer (appending to the cache)
+// and leaves the residual stream in ws.x; the head turns rows of it into logits or greedy picks.
+struct b200nn_lm {
     b200nn_ctx *ctx = nullptr;
+    virtual ~b200nn_lm() = default;
+    virtual const char *family() const = 0;
+    virtual int vocab() const = 0;
+    virtual int width() const = 0;
+    virtual int n_layer() const = 0;
+    virtual size_t max_positions() const { return 0; } // 0: the cache's capacity is the only limit
+    virtual long long eos() const { return -1; }       // end-of-text token, -1: none
+    virtual int cache_init(size_t batch, size_t cap, b200nn_kvcache *c) = 0;
+    virtual int workspace_init(size_t rows, size_t logit_rows, Workspace *ws) = 0;
+    // Prompt portions: the rows of all entries, in order (ids on the host); no entry longer than
+    // b200nn_kvcache::portion (0: no limit).  Does not advance the cache's lengths.
+    virtual int pass_prompt(Workspace &ws, b200nn_kvcache &kv, const std::vector<PassEntry> &entries, const uint32_t *ids_host) = 0;
+    // One token of every sequence of the cache: ws.tok at the device-side position *pos_ptr.
+    virtual int pass_decode(Workspace &ws, b200nn_kvcache &kv, const int *pos_ptr, StepProfile *prof) = 0;
+    virtual int head(Workspace &ws, const float *x, int rows, StepProfile *prof) = 0; // -> ws.logits
+    virtual int head_pick(Workspace &ws, const float *x, int rows, bool keep_last, bool tokens_only, uint32_t *tok_out,
+                          StepProfile *prof) = 0;
+};
+
+struct b200nn_gpt2 : b200nn_lm {
+    const char *family() const override { return "gpt2"; }
+    int vocab() const override { return cfg.vocab_size; }
+    int width() const override { return cfg.n_embd; }
+    int n_layer() const override { return cfg.n_layer; }
+    size_t max_positions() const override { return (size_t)cfg.n_positions; }
+    long long eos() const override { return 50256; }
+    int cache_init(size_t batch, size_t cap, b200nn_kvcache *c) override;
+    int workspace_init(size_t rows, size_t logit_rows, Workspace *ws) override;
+    int pass_prompt(Workspace &ws, b200nn_kvcache &kv, const std::vector<PassEntry> &entries, const uint32_t *ids_host) override;
+    int pass_decode(Workspace &ws, b200nn_kvcache &kv, const int *pos_ptr, StepProfile *prof) override;
+    int head(Workspace &ws, const float *x, int rows, StepProfile *prof) override;
+    int head_pick(Workspace &ws, const float *x, int rows, bool keep_last, bool tokens_only, uint32_t *tok_out,
+                  StepProfile *prof) override;
     b200nn_gpt2_config cfg{};
     uint32_t flags = 0;
     bool int4 = false;
@@ -66,11 +114,37 @@ struct b200nn_gpt2 {
     int act() const { return (flags & B200NN_GELU_SIGMOID) ? B200NN_ACT_GELU_SIGMOID : B200NN_ACT_GELU_TANH; }
 };
 
+// What one run of a hybrid model's layer keeps per sequence slot (a layer that shares another's weights has a
+// record of its own).
+struct LayerState {
+    // latent attention: [slot][ring][ld] rows of (latent, rotated key part); position p lives in row p % ring
+    std::shared_ptr<DevBuf> latent;
+    int ring = 0;
+    // delta rule: [slot][head][dim][vdim] f32 state, [slot][taps][channel] f32 convolution inputs (position
+    // p in row p % taps)
+    std::shared_ptr<DevBuf> state, conv;
+};
+
+// KV cache / state manager: `batch` sequence slots of up to `cap` positions.  Lockstep use (decode session,
+// forward_cached) advances all slots together and keeps `len`; the serving step (b200nn_lm_step) keeps a
+// length per slot and hands slots out and back.
 struct b200nn_kvcache {
-    b200nn_gpt2 *m = nullptr;
+    b200nn_lm *m = nullptr;
     size_t batch = 0, cap = 0, len = 0;
+    size_t portion = 0;          // most new tokens of one sequence in a pass (0: no limit)
+    std::vector<size_t> slot_len; // serving: positions held per slot
+    std::vector<char> slot_used;
+    std::unique_ptr<Workspace> ws; // serving: activation buffers, grown on demand
+    // GPT-2
+    size_t n_head = 0;
     std::shared_ptr<DevBuf> k, v; // [layer][seq][head][cap][64] fp16
-    size_t layer_stride() const { return batch * (size_t)m->cfg.n_head * cap * 64; }
+    // hybrid models: one record per layer run, and one angle table [cap][pair] (cos, sin) per rotation in use
+    std::vector<LayerState> layers;
+    std::vector<std::shared_ptr<DevBuf>> rope;
+    b200nn_kvcache();
+    ~b200nn_kvcache();
+    b200nn_kvcache(const b200nn_kvcache &) = delete;
+    size_t layer_stride() const { return batch * n_head * cap * 64; }
     __half *kl(int l) const { return static_cast<__half *>(k->p) + (size_t)l * layer_stride(); }
     __half *vl(int l) const { return static_cast<__half *>(v->p) + (size_t)l * layer_stride(); }
 };
@@ -86,6 +160,8 @@ struct Workspace {
     std::shared_ptr<DevBuf> ln_stats;
     int ln_nt = 0;
     float *ln_slot(int i) const { return static_cast<float *>(ln_stats->p) + (size_t)i * rows * ln_nt * 2; }
+    // hybrid models (sizes in hybrid.cu)
+    std::shared_ptr<DevBuf> proj, gate, cq, qlat, olat, heads, dstep, lin, kvx, part, meta;
 };
 int workspace_alloc(b200nn_gpt2 *m, size_t rows, size_t logit_rows, Workspace *ws);
 
@@ -130,8 +206,18 @@ int run_head_pick(b200nn_gpt2 *m, Workspace &ws, const float *x, int rows, bool 
 int run_head(b200nn_gpt2 *m, Workspace &ws, const float *x, int rows, bool act_half, StepProfile *prof);
 bool model_act_half(const b200nn_gpt2 *m, int rows);
 
+inline void prof_mark(b200nn_ctx *ctx, StepProfile *p, int fam) {
+    if (!p) return;
+    cudaEvent_t e;
+    cudaEventCreate(&e);
+    cudaEventRecord(e, ctx->stream);
+    p->ev.push_back(e);
+    p->fam.push_back(fam);
+}
+
 struct b200nn_session {
-    b200nn_gpt2 *m = nullptr;
+    b200nn_lm *m = nullptr;
+    b200nn_gpt2 *gpt2 = nullptr; // the same model when it is of that family
     size_t batch = 0, cap = 0, hist_cap = 0;
     uint32_t flags = 0;
     b200nn_kvcache kv;

@@ -315,8 +315,9 @@ int int4_weight_ln_fold(b200nn_ctx *ctx, const Int4Weight &w, const float *g_dev
 }
 
 int f32_weight_upload(b200nn_ctx *ctx, const float *wsrc, bool is_out_in, const float *bias, size_t K, size_t N,
-                      F32Weight *w) {
+                      F32Weight *w, bool exact) {
     if (K == 0 || N == 0) return set_error(ctx, B200NN_ERR_SHAPE, "Linear: empty weight");
+    w->exact = exact;
     w->K = (int)K;
     w->N = (int)N;
     if (is_out_in) { // [N,K] -> [K,N]
@@ -335,7 +336,7 @@ int f32_weight_upload(b200nn_ctx *ctx, const float *wsrc, bool is_out_in, const 
     // then lo[N,K] = the rounded remainder w - hi.  Skipped when a value would overflow fp16 or the
     // row stride would not be a multiple of 16 bytes.
     w->w_nk_h.reset();
-    if (K % 8 == 0) {
+    if (K % 8 == 0 && !exact) {
         std::vector<__half> h(2 * K * N);
         __half *hp = h.data(), *lp = h.data() + K * N;
         std::atomic<int> too_large{0};
@@ -353,5 +354,33 @@ int f32_weight_upload(b200nn_ctx *ctx, const float *wsrc, bool is_out_in, const 
         });
         if (!too_large.load()) TRY(upload(ctx, h.data(), h.size() * sizeof(__half), &w->w_nk_h));
     }
+    return B200NN_OK;
+}
+
+int b16_weight_upload(b200nn_ctx *ctx, const float *w_nk, size_t K, size_t N, B16Weight *w) {
+    if (K == 0 || N == 0 || K % 8 != 0) return set_error(ctx, B200NN_ERR_SHAPE, "bf16 Linear: K must be a positive multiple of 8");
+    w->K = (int)K;
+    w->N = (int)N;
+    std::vector<__nv_bfloat16> h(K * N);
+    __nv_bfloat16 *hp = h.data();
+    parallel_for(N, [=](size_t n0, size_t n1) {
+        for (size_t i = n0 * K; i < n1 * K; ++i) hp[i] = __float2bfloat16_rn(w_nk[i]);
+    });
+    return upload(ctx, h.data(), h.size() * sizeof(__nv_bfloat16), &w->w_nk);
+}
+
+int b16_grouped_weight_upload(b200nn_ctx *ctx, const float *w_gnk, size_t groups, size_t Ng, size_t Kg, size_t x_stride,
+                              size_t out_stride, B16Weight *w) {
+    if (Ng % 4 != 0 || out_stride % 4 != 0 || x_stride % 8 != 0)
+        return set_error(ctx, B200NN_ERR_SHAPE, "grouped bf16 Linear: group widths must keep 16-byte alignment");
+    const size_t tiles = (Ng + TILE_N - 1) / TILE_N, rows = tiles * TILE_N;
+    std::vector<float> padded(groups * rows * Kg, 0.0f);
+    for (size_t g = 0; g < groups; ++g) std::copy(w_gnk + g * Ng * Kg, w_gnk + (g + 1) * Ng * Kg, padded.begin() + g * rows * Kg);
+    TRY(b16_weight_upload(ctx, padded.data(), Kg, groups * rows, w));
+    w->groups = (int)groups;
+    w->group_n = (int)Ng;
+    w->group_tiles = (int)tiles;
+    w->group_kx = (int)x_stride;
+    w->group_stride = (int)out_stride;
     return B200NN_OK;
 }

@@ -13,6 +13,7 @@
 #include <cstring>
 #include <map>
 
+#include "json.h"
 #include "model.h"
 
 namespace {
@@ -29,87 +30,6 @@ int st_fail(int code, const std::string &msg) {
     g_st_error = msg;
     return code;
 }
-
-// ---- a JSON reader sufficient for the header: objects, arrays, strings, non-negative integers ----
-struct Json {
-    const char *p, *e;
-    bool ok = true;
-    void ws() {
-        while (p < e && (*p == ' ' || *p == '\n' || *p == '\t' || *p == '\r')) ++p;
-    }
-    bool eat(char c) {
-        ws();
-        if (p < e && *p == c) { ++p; return true; }
-        return false;
-    }
-    bool str(std::string &out) {
-        ws();
-        if (p >= e || *p != '"') return ok = false;
-        ++p;
-        out.clear();
-        while (p < e && *p != '"') {
-            if (*p == '\\') {
-                if (++p >= e) return ok = false;
-                switch (*p) {
-                    case 'n': out += '\n'; break;
-                    case 't': out += '\t'; break;
-                    case 'r': out += '\r'; break;
-                    case 'b': out += '\b'; break;
-                    case 'f': out += '\f'; break;
-                    case 'u': { // basic multilingual plane -> UTF-8
-                        if (e - p < 5) return ok = false;
-                        unsigned v = 0;
-                        for (int i = 1; i <= 4; ++i) {
-                            const char h = p[i];
-                            v <<= 4;
-                            if (h >= '0' && h <= '9') v |= h - '0';
-                            else if (h >= 'a' && h <= 'f') v |= h - 'a' + 10;
-                            else if (h >= 'A' && h <= 'F') v |= h - 'A' + 10;
-                            else return ok = false;
-                        }
-                        p += 4;
-                        if (v < 0x80) out += (char)v;
-                        else if (v < 0x800) { out += (char)(0xC0 | (v >> 6)); out += (char)(0x80 | (v & 0x3F)); }
-                        else { out += (char)(0xE0 | (v >> 12)); out += (char)(0x80 | ((v >> 6) & 0x3F)); out += (char)(0x80 | (v & 0x3F)); }
-                        break;
-                    }
-                    default: out += *p; // \" \\ \/
-                }
-                ++p;
-            } else {
-                out += *p++;
-            }
-        }
-        if (p >= e) return ok = false;
-        ++p;
-        return true;
-    }
-    bool uint(size_t &v) {
-        ws();
-        if (p >= e || *p < '0' || *p > '9') return ok = false;
-        v = 0;
-        while (p < e && *p >= '0' && *p <= '9') v = v * 10 + (size_t)(*p++ - '0');
-        return true;
-    }
-    bool skip() { // any value
-        ws();
-        if (p >= e) return ok = false;
-        if (*p == '"') { std::string s; return str(s); }
-        if (*p == '{' || *p == '[') {
-            const char close = *p == '{' ? '}' : ']';
-            const bool obj = *p == '{';
-            ++p;
-            if (eat(close)) return true;
-            do {
-                if (obj) { std::string k; if (!str(k) || !eat(':')) return ok = false; }
-                if (!skip()) return false;
-            } while (eat(','));
-            return eat(close) ? true : (ok = false);
-        }
-        while (p < e && *p != ',' && *p != '}' && *p != ']') ++p; // number / true / false / null
-        return true;
-    }
-};
 
 size_t dtype_size(const std::string &d) {
     if (d == "F64" || d == "I64" || d == "U64") return 8;

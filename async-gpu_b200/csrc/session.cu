@@ -4,21 +4,21 @@
 
 #include "model.h"
 
-static int kv_init(b200nn_gpt2 *m, size_t batch, size_t cap, b200nn_kvcache *c) {
+static int kv_init(b200nn_lm *m, size_t batch, size_t cap, b200nn_kvcache *c) {
     if (!batch || !cap) return set_error(m->ctx, B200NN_ERR_SHAPE, "KvCache: batch and capacity must be positive");
-    if (cap > (size_t)m->cfg.n_positions)
-        return set_error(m->ctx, B200NN_ERR_DIM, "KvCache: capacity exceeds n_positions");
     c->m = m;
     c->batch = batch;
     c->cap = cap;
     c->len = 0;
-    size_t bytes = (size_t)m->cfg.n_layer * batch * m->cfg.n_embd * cap * sizeof(__half);
-    TRY(dev_alloc(m->ctx, bytes, &c->k));
-    TRY(dev_alloc(m->ctx, bytes, &c->v));
-    return B200NN_OK;
+    c->slot_len.assign(batch, 0);
+    c->slot_used.assign(batch, 0);
+    return m->cache_init(batch, cap, c);
 }
 
 extern "C" int32_t b200nn_kvcache_create(b200nn_gpt2 *m, size_t batch, size_t capacity, b200nn_kvcache **out) {
+    return b200nn_lm_cache_create(m, batch, capacity, out);
+}
+extern "C" int32_t b200nn_lm_cache_create(b200nn_lm *m, size_t batch, size_t capacity, b200nn_kvcache **out) {
     if (!m || !out) return B200NN_ERR_ARG;
     auto c = std::unique_ptr<b200nn_kvcache>(new b200nn_kvcache());
     TRY(kv_init(m, batch, capacity, c.get()));
@@ -29,13 +29,14 @@ extern "C" size_t b200nn_kvcache_len(const b200nn_kvcache *c) { return c ? c->le
 extern "C" int32_t b200nn_kvcache_reset(b200nn_kvcache *c) {
     if (!c) return B200NN_ERR_ARG;
     c->len = 0;
+    std::fill(c->slot_len.begin(), c->slot_len.end(), 0);
     return B200NN_OK;
 }
 extern "C" void b200nn_kvcache_destroy(b200nn_kvcache *c) { delete c; }
 
-static int check_ids(b200nn_gpt2 *m, const uint32_t *ids, size_t n) {
+static int check_ids(b200nn_lm *m, const uint32_t *ids, size_t n) {
     for (size_t i = 0; i < n; ++i)
-        if (ids[i] >= (uint32_t)m->cfg.vocab_size)
+        if (ids[i] >= (uint32_t)m->vocab())
             return set_error(m->ctx, B200NN_ERR_DIM, "token id out of range for vocab_size");
     return B200NN_OK;
 }
@@ -118,23 +119,28 @@ static constexpr size_t PREFILL_ROWS = 16384; // rows per prefill pass (bounds t
 
 extern "C" int32_t b200nn_session_create(b200nn_gpt2 *m, size_t batch, size_t capacity, uint32_t flags,
                                          b200nn_session **out) {
+    return b200nn_lm_session_create(m, batch, capacity, flags, out);
+}
+extern "C" int32_t b200nn_lm_session_create(b200nn_lm *m, size_t batch, size_t capacity, uint32_t flags,
+                                            b200nn_session **out) {
     if (!m || !out) return B200NN_ERR_ARG;
     b200nn_ctx *ctx = m->ctx;
     CK(ctx, cudaSetDevice(ctx->device));
     auto s = std::unique_ptr<b200nn_session>(new b200nn_session());
     s->m = m;
+    s->gpt2 = dynamic_cast<b200nn_gpt2 *>(m);
     s->batch = batch;
     s->cap = capacity;
     s->hist_cap = capacity;
     s->flags = flags;
     TRY(kv_init(m, batch, capacity, &s->kv));
-    TRY(workspace_alloc(m, batch, batch, &s->ws_step));
+    TRY(m->workspace_init(batch, batch, &s->ws_step));
     TRY(dev_alloc(ctx, 2 * sizeof(int), &s->counters));
     CK(ctx, cudaMemsetAsync(s->counters->p, 0, 2 * sizeof(int), ctx->stream));
     TRY(dev_alloc(ctx, batch * s->hist_cap * 4, &s->history));
     CK(ctx, cudaMemsetAsync(s->history->p, 0, batch * s->hist_cap * 4, ctx->stream));
-    if (model_ln_fold_supported(m, (int)batch)) TRY(model_prepare_ln_fold(m, &s->ws_step));
-    if (decode_persistent_supported(m, (int)batch)) {
+    if (s->gpt2 && model_ln_fold_supported(s->gpt2, (int)batch)) TRY(model_prepare_ln_fold(s->gpt2, &s->ws_step));
+    if (s->gpt2 && decode_persistent_supported(s->gpt2, (int)batch)) {
         TRY(decode_persistent_prepare(s.get()));
         s->persist = true;
     }
@@ -158,45 +164,45 @@ static int set_counters(b200nn_session *s, int position, int step) {
 
 extern "C" int32_t b200nn_session_prefill(b200nn_session *s, const uint32_t *prompts_host, size_t prompt_len) {
     if (!s || !prompts_host) return B200NN_ERR_ARG;
-    b200nn_gpt2 *m = s->m;
+    b200nn_lm *m = s->m;
     b200nn_ctx *ctx = m->ctx;
     if (prompt_len == 0 || prompt_len >= s->cap)
         return set_error(ctx, B200NN_ERR_DIM, "prefill: prompt_len must be in [1, capacity)");
     CK(ctx, cudaSetDevice(ctx->device));
-    const int d = m->cfg.n_embd;
-    size_t seqs_per_pass = std::max<size_t>(1, PREFILL_ROWS / prompt_len);
+    TRY(check_ids(m, prompts_host, s->batch * prompt_len));
+    const int d = m->width();
+    // a prompt longer than the cache takes in one pass goes through in portions
+    const size_t part = s->kv.portion ? std::min(prompt_len, s->kv.portion) : prompt_len;
+    size_t seqs_per_pass = std::max<size_t>(1, PREFILL_ROWS / part);
     seqs_per_pass = std::min(seqs_per_pass, s->batch);
-    if (s->ws_prefill.rows < seqs_per_pass * prompt_len || s->ws_prefill.logit_rows < 1) {
+    if (s->ws_prefill.rows < seqs_per_pass * part || s->ws_prefill.logit_rows < 1) {
         s->ws_prefill = Workspace();
-        TRY(workspace_alloc(m, seqs_per_pass * prompt_len, 1, &s->ws_prefill));
+        TRY(m->workspace_init(seqs_per_pass * part, 1, &s->ws_prefill));
     }
     s->kv.len = 0;
     float *last_x = (float *)s->ws_step.last_x->p;
+    std::vector<PassEntry> entries;
+    std::vector<uint32_t> ids;
     for (size_t b0 = 0; b0 < s->batch; b0 += seqs_per_pass) {
-        size_t nb = std::min(seqs_per_pass, s->batch - b0);
-        // a view of the cache that starts at sequence b0
-        b200nn_kvcache view;
-        view.m = m;
-        view.batch = s->batch; // layer stride of the full cache
-        view.cap = s->cap;
-        view.len = 0;
-        view.k = std::make_shared<DevBuf>();
-        view.v = std::make_shared<DevBuf>();
-        size_t seq_off = b0 * (size_t)m->cfg.n_head * s->cap * 64;
-        view.k->p = (__half *)s->kv.k->p + seq_off;
-        view.v->p = (__half *)s->kv.v->p + seq_off;
-        bool ah = model_act_half(m, (int)(nb * prompt_len));
-        int rc = forward_rows(m, s->ws_prefill, view, prompts_host + b0 * prompt_len, (int)nb, (int)prompt_len, ah);
-        view.k->p = nullptr; // borrowed pointers: nothing to free
-        view.v->p = nullptr;
-        TRY(rc);
-        TRY(launch_gather_last_rows(ctx, (const float *)s->ws_prefill.x->p, (int)nb, (int)prompt_len, d,
-                                    last_x + b0 * d));
+        const size_t nb = std::min(seqs_per_pass, s->batch - b0);
+        for (size_t p0 = 0; p0 < prompt_len; p0 += part) {
+            const size_t n = std::min(part, prompt_len - p0);
+            const uint32_t *src = prompts_host + b0 * prompt_len;
+            entries.clear();
+            for (size_t i = 0; i < nb; ++i) entries.push_back(PassEntry{(int)(b0 + i), (int)p0, (int)n});
+            if (n != prompt_len) {
+                ids.resize(nb * n);
+                for (size_t i = 0; i < nb; ++i) memcpy(&ids[i * n], src + i * prompt_len + p0, n * 4);
+                src = ids.data();
+            }
+            TRY(m->pass_prompt(s->ws_prefill, s->kv, entries, src));
+            if (p0 + n == prompt_len)
+                TRY(launch_gather_last_rows(ctx, (const float *)s->ws_prefill.x->p, (int)nb, (int)n, d, last_x + b0 * d));
+        }
     }
     s->kv.len = prompt_len;
-    bool ah = model_act_half(m, (int)s->batch);
-    TRY(run_head_pick(m, s->ws_step, last_x, (int)s->batch, ah, (s->flags & B200NN_ARGMAX_LAST) != 0,
-                      (s->flags & B200NN_TOKENS_ONLY) != 0, (uint32_t *)s->ws_step.tok->p, nullptr));
+    TRY(m->head_pick(s->ws_step, last_x, (int)s->batch, (s->flags & B200NN_ARGMAX_LAST) != 0,
+                     (s->flags & B200NN_TOKENS_ONLY) != 0, (uint32_t *)s->ws_step.tok->p, nullptr));
     TRY(set_counters(s, (int)prompt_len - 1, 0));
     // record: history[0] = first token, step = 1, position = prompt_len
     TRY(launch_record_tokens(ctx, (const uint32_t *)s->ws_step.tok->p, (int)s->batch, (uint32_t *)s->history->p,
@@ -208,55 +214,30 @@ extern "C" int32_t b200nn_session_prefill(b200nn_session *s, const uint32_t *pro
 }
 
 // One greedy decode step for every sequence: embed the current tokens at the device-side
-// position, run the blocks (K,V appended in the QKV epilogue), LM head, argmax, record.
+// position, run the layers (the cache is appended to on the way), LM head, argmax, record.
 static int decode_step(b200nn_session *s, StepProfile *prof) {
-    b200nn_gpt2 *m = s->m;
+    b200nn_lm *m = s->m;
     b200nn_ctx *ctx = m->ctx;
-    const int B = (int)s->batch, d = m->cfg.n_embd;
+    const int B = (int)s->batch;
     Workspace &ws = s->ws_step;
-    bool ah = model_act_half(m, B);
-    const bool persistent = s->persist && ctx->persist;
-    const bool fold = !persistent && ws.ln_stats && ctx->ln_fold && model_ln_fold_supported(m, B);
-    if (fold)
-        TRY(launch_embedding_ln(ctx, (const uint32_t *)ws.tok->p, (const float *)m->wte->p, (const float *)m->wpe->p, B, d,
-                                s->pos_ptr(), m->cfg.vocab_size, m->cfg.n_positions, (float *)ws.x->p,
-                                (const float *)m->blocks[0].ln1_g->p, (__half *)ws.ln->p, ws.ln_slot(0), ws.ln_nt));
-    else
-        TRY(launch_embedding(ctx, (const uint32_t *)ws.tok->p, (const float *)m->wte->p, (const float *)m->wpe->p, B, d, 1,
-                             s->pos_ptr(), 0, m->cfg.vocab_size, m->cfg.n_positions, (float *)ws.x->p));
-    if (prof) {
-        cudaEvent_t e;
-        cudaEventCreate(&e);
-        cudaEventRecord(e, ctx->stream);
-        prof->ev.push_back(e);
-        prof->fam.push_back(B200NN_PROF_EMBED);
-    }
-    if (persistent) {
+    if (s->persist && ctx->persist) {
+        b200nn_gpt2 *g = s->gpt2;
+        TRY(launch_embedding(ctx, (const uint32_t *)ws.tok->p, (const float *)g->wte->p, (const float *)g->wpe->p, B,
+                             g->cfg.n_embd, 1, s->pos_ptr(), 0, g->cfg.vocab_size, g->cfg.n_positions, (float *)ws.x->p));
+        prof_mark(ctx, prof, B200NN_PROF_EMBED);
         // every transformer block in one cooperative launch; with `prof` its phases are timed inside the
         // kernel and the launch as a whole is booked under the attention family's event slot
         if (prof) CK(ctx, cudaMemsetAsync((char *)s->pd_sync->p + 64, 0, 128, ctx->stream));
         TRY(launch_decode_layers(s, prof != nullptr));
-        if (prof) {
-            cudaEvent_t e;
-            cudaEventCreate(&e);
-            cudaEventRecord(e, ctx->stream);
-            prof->ev.push_back(e);
-            prof->fam.push_back(-1); // split by the in-kernel phase times afterwards
-        }
+        prof_mark(ctx, prof, -1); // split by the in-kernel phase times afterwards
     } else {
-        TRY(run_blocks(m, ws, s->kv, B, 1, s->pos_ptr(), 0, ah, prof, fold));
+        TRY(m->pass_decode(ws, s->kv, s->pos_ptr(), prof));
     }
-    TRY(run_head_pick(m, ws, (const float *)ws.x->p, B, ah, (s->flags & B200NN_ARGMAX_LAST) != 0,
-                      (s->flags & B200NN_TOKENS_ONLY) != 0, (uint32_t *)ws.tok->p, prof));
+    TRY(m->head_pick(ws, (const float *)ws.x->p, B, (s->flags & B200NN_ARGMAX_LAST) != 0,
+                     (s->flags & B200NN_TOKENS_ONLY) != 0, (uint32_t *)ws.tok->p, prof));
     TRY(launch_record_tokens(ctx, (const uint32_t *)ws.tok->p, B, (uint32_t *)s->history->p, (int)s->hist_cap,
                              s->step_ptr(), s->pos_ptr()));
-    if (prof) {
-        cudaEvent_t e;
-        cudaEventCreate(&e);
-        cudaEventRecord(e, ctx->stream);
-        prof->ev.push_back(e);
-        prof->fam.push_back(B200NN_PROF_ARGMAX);
-    }
+    prof_mark(ctx, prof, B200NN_PROF_ARGMAX);
     return B200NN_OK;
 }
 
@@ -344,14 +325,14 @@ extern "C" int32_t b200nn_session_logits(b200nn_session *s, float *out) {
     if (s->flags & B200NN_TOKENS_ONLY)
         return set_error(ctx, B200NN_ERR_UNSUPPORTED, "session_logits: the session was created with B200NN_TOKENS_ONLY");
     CK(ctx, cudaSetDevice(ctx->device));
-    CK(ctx, cudaMemcpyAsync(out, s->ws_step.logits->p, s->batch * (size_t)s->m->cfg.vocab_size * 4,
+    CK(ctx, cudaMemcpyAsync(out, s->ws_step.logits->p, s->batch * (size_t)s->m->vocab() * 4,
                             cudaMemcpyDeviceToHost, ctx->stream));
     return stream_sync_check(ctx);
 }
 
 extern "C" int32_t b200nn_session_profile_step(b200nn_session *s, float *times_ms, uint64_t *linear_bytes) {
     if (!s || !times_ms) return B200NN_ERR_ARG;
-    b200nn_gpt2 *m = s->m;
+    b200nn_lm *m = s->m;
     b200nn_ctx *ctx = m->ctx;
     if (!s->prefilled) return set_error(ctx, B200NN_ERR_ARG, "profile_step before prefill");
     if (s->position + 1 > s->cap) return set_error(ctx, B200NN_ERR_DIM, "profile_step: capacity exceeded");
@@ -389,12 +370,13 @@ extern "C" int32_t b200nn_session_profile_step(b200nn_session *s, float *times_m
     s->position += 1;
     s->steps_done += 1;
     s->kv.len = s->position;
-    if (linear_bytes) {
+    if (linear_bytes && !s->gpt2) *linear_bytes = 0; // accounted for by the caller, who knows the layers
+    else if (linear_bytes) {
         // algorithmic bytes of the block Linears in one step: weights + scales + bias, the
         // activations read and the outputs written (LM head reported under its own family)
-        bool ah = model_act_half(m, (int)s->batch);
-        size_t ab = ah ? 2 : 4, B = s->batch, d = m->cfg.n_embd, t = 0;
-        for (const BlockW &b : m->blocks) {
+        bool ah = model_act_half(s->gpt2, (int)s->batch);
+        size_t ab = ah ? 2 : 4, B = s->batch, d = m->width(), t = 0;
+        for (const BlockW &b : s->gpt2->blocks) {
             t += b.qkv.weight_bytes() + B * d * ab + B * 3 * d * 2;       // q + K,V as fp16 / act dtype
             t += b.proj.weight_bytes() + B * d * ab + 2 * B * d * 4;      // residual read + write
             t += b.fc.weight_bytes() + B * d * ab + B * 4 * d * ab;
@@ -408,8 +390,9 @@ extern "C" int32_t b200nn_session_profile_step(b200nn_session *s, float *times_m
 extern "C" int32_t b200nn_session_time_family(b200nn_session *s, int32_t family, int32_t reps, float *ms_total,
                                               uint64_t *launches) {
     if (!s || !ms_total || reps <= 0) return B200NN_ERR_ARG;
-    b200nn_gpt2 *m = s->m;
-    b200nn_ctx *ctx = m->ctx;
+    b200nn_gpt2 *m = s->gpt2;
+    b200nn_ctx *ctx = s->m->ctx;
+    if (!m) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "time_family: GPT-2 sessions only");
     if (!s->prefilled) return set_error(ctx, B200NN_ERR_ARG, "time_family before prefill");
     if (family != B200NN_PROF_LAYERNORM && family != B200NN_PROF_LINEAR && family != B200NN_PROF_ATTENTION &&
         family != B200NN_PROF_LM_HEAD)
@@ -472,10 +455,14 @@ extern "C" int32_t b200nn_session_time_family(b200nn_session *s, int32_t family,
 extern "C" int32_t b200nn_gpt2_generate_batch(b200nn_gpt2 *m, const uint32_t *prompts, size_t batch,
                                               size_t prompt_len, size_t max_new, uint32_t flags,
                                               uint32_t *out_tokens, size_t *out_lens) {
+    return b200nn_lm_generate_batch(m, prompts, batch, prompt_len, max_new, flags, out_tokens, out_lens);
+}
+extern "C" int32_t b200nn_lm_generate_batch(b200nn_lm *m, const uint32_t *prompts, size_t batch, size_t prompt_len,
+                                            size_t max_new, uint32_t flags, uint32_t *out_tokens, size_t *out_lens) {
     if (!m || !prompts || !out_tokens) return B200NN_ERR_ARG;
     b200nn_ctx *ctx = m->ctx;
     if (batch == 0 || prompt_len == 0) return set_error(ctx, B200NN_ERR_SHAPE, "generate: empty batch or prompt");
-    if (prompt_len + max_new > (size_t)m->cfg.n_positions)
+    if (m->max_positions() && prompt_len + max_new > m->max_positions())
         return set_error(ctx, B200NN_ERR_DIM, "generate: prompt_len + max_new exceeds n_positions");
     const size_t stride = prompt_len + max_new;
     for (size_t b = 0; b < batch; ++b) {
@@ -484,7 +471,7 @@ extern "C" int32_t b200nn_gpt2_generate_batch(b200nn_gpt2 *m, const uint32_t *pr
     }
     if (max_new == 0) return B200NN_OK;
     b200nn_session *s = nullptr;
-    TRY(b200nn_session_create(m, batch, stride, flags | B200NN_TOKENS_ONLY, &s)); // greedy tokens are all that is returned
+    TRY(b200nn_lm_session_create(m, batch, stride, flags | B200NN_TOKENS_ONLY, &s)); // greedy tokens are all that is returned
     std::unique_ptr<b200nn_session, void (*)(b200nn_session *)> guard(s, b200nn_session_destroy);
     TRY(b200nn_session_prefill(s, prompts, prompt_len));
     TRY(b200nn_session_step(s, max_new - 1));
@@ -493,9 +480,9 @@ extern "C" int32_t b200nn_gpt2_generate_batch(b200nn_gpt2 *m, const uint32_t *pr
     TRY(b200nn_session_tokens(s, gen.data(), max_new, &n));
     for (size_t b = 0; b < batch; ++b) {
         size_t len = n;
-        if (flags & B200NN_STOP_ON_EOS) // stop before appending <|endoftext|> (gpt2.rs:698-700)
+        if ((flags & B200NN_STOP_ON_EOS) && m->eos() >= 0) // stop before appending <|endoftext|> (gpt2.rs:698-700)
             for (size_t i = 0; i < n; ++i)
-                if (gen[b * max_new + i] == 50256u) { len = i; break; }
+                if (gen[b * max_new + i] == (uint32_t)m->eos()) { len = i; break; }
         memcpy(out_tokens + b * stride + prompt_len, gen.data() + b * max_new, len * 4);
         if (out_lens) out_lens[b] = prompt_len + len;
     }

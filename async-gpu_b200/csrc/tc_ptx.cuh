@@ -165,6 +165,8 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mn64(uint32_t smem_addr) { r
 __host__ __device__ constexpr uint32_t umma_idesc_f16(int M, int N) {
     return (1u << 4) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
 }
+// Format bits to add for bfloat16 A and B (a_format = b_format = 1).
+static constexpr uint32_t UMMA_BF16 = (1u << 7) | (1u << 10);
 // The same with the B operand MN-major (bit 16): B[k][n] lies with n contiguous in shared memory.
 __host__ __device__ constexpr uint32_t umma_idesc_f16_bmn(int M, int N) { return umma_idesc_f16(M, N) | (1u << 16); }
 // D[tmem] (+)= A[smem] * B[smem]; issued by one thread.

@@ -47,7 +47,7 @@ fn main() {
             .arg("-o").arg(&obj));
         objects.push(obj);
     }
-    for h in ["common.h", "model.h", "device_utils.cuh", "tc_ptx.cuh"] {
+    for h in ["common.h", "model.h", "hybrid.h", "json.h", "device_utils.cuh", "tc_ptx.cuh"] {
         println!("cargo:rerun-if-changed={}", csrc.join(h).display());
     }
     let lib = out.join("libb200nn.so");

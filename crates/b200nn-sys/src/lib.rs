@@ -36,6 +36,7 @@ pub const B200NN_ARGMAX_LAST: u32 = 1 << 2;
 pub const B200NN_STOP_ON_EOS: u32 = 1 << 3;
 pub const B200NN_TOKENS_ONLY: u32 = 1 << 4;
 pub const B200NN_WEIGHTS_OUT_IN: u32 = 1 << 5;
+pub const B200NN_LM_F32: u32 = 1 << 6;
 
 /// Kernel families of `b200nn_session_profile_step` / `b200nn_session_time_family`.
 pub const B200NN_PROF_EMBED: i32 = 0;
@@ -44,7 +45,8 @@ pub const B200NN_PROF_LINEAR: i32 = 2;
 pub const B200NN_PROF_ATTENTION: i32 = 3;
 pub const B200NN_PROF_LM_HEAD: i32 = 4;
 pub const B200NN_PROF_ARGMAX: i32 = 5;
-pub const B200NN_PROF_COUNT: i32 = 6;
+pub const B200NN_PROF_RECURRENCE: i32 = 6;
+pub const B200NN_PROF_COUNT: i32 = 7;
 
 macro_rules! opaque {
     ($($name:ident),* $(,)?) => {
@@ -58,6 +60,7 @@ macro_rules! opaque {
 }
 opaque!(
     b200nn_ctx,
+    b200nn_lm,
     b200nn_tensor,
     b200nn_linear,
     b200nn_int4_linear,
@@ -82,6 +85,17 @@ pub struct b200nn_gpt2_config {
     pub vocab_size: i32,
     pub n_positions: i32,
     pub layer_norm_epsilon: f32,
+}
+
+/// What a model of any family tells of itself (`n_positions` 0: no limit of its own, `eos_token` -1: none).
+#[repr(C)]
+#[derive(Clone, Copy, Debug, PartialEq)]
+pub struct b200nn_lm_info {
+    pub n_layer: i32,
+    pub width: i32,
+    pub vocab_size: i32,
+    pub n_positions: i32,
+    pub eos_token: i32,
 }
 
 /// `TransformerLayerWeights` (model.rs:112-139): host f32, dense weights in Conv1D layout [in,out].
@@ -670,6 +684,63 @@ extern "C" {
         int4_group: usize,
         flags: u32,
         out: *mut *mut b200nn_gpt2,
+    ) -> i32;
+    pub fn b200nn_lm_create(
+        ctx: *mut b200nn_ctx,
+        config_json: *const c_char,
+        n_tensors: usize,
+        names: *const *const c_char,
+        data: *const *const f32,
+        numels: *const usize,
+        flags: u32,
+        out: *mut *mut b200nn_lm,
+    ) -> i32;
+    pub fn b200nn_lm_load(ctx: *mut b200nn_ctx, dir: *const c_char, flags: u32, out: *mut *mut b200nn_lm) -> i32;
+    pub fn b200nn_gpt2_as_lm(m: *mut b200nn_gpt2) -> *mut b200nn_lm;
+    pub fn b200nn_lm_destroy(m: *mut b200nn_lm);
+    pub fn b200nn_lm_get_info(m: *const b200nn_lm, out: *mut b200nn_lm_info) -> i32;
+    pub fn b200nn_lm_family(m: *const b200nn_lm) -> *const c_char;
+    pub fn b200nn_lm_cache_create(m: *mut b200nn_lm, slots: usize, capacity: usize, out: *mut *mut b200nn_kvcache) -> i32;
+    pub fn b200nn_lm_session_create(
+        m: *mut b200nn_lm,
+        batch: usize,
+        capacity: usize,
+        flags: u32,
+        out: *mut *mut b200nn_session,
+    ) -> i32;
+    pub fn b200nn_lm_generate_batch(
+        m: *mut b200nn_lm,
+        prompts: *const u32,
+        batch: usize,
+        prompt_len: usize,
+        max_new: usize,
+        flags: u32,
+        out_tokens: *mut u32,
+        out_lens: *mut usize,
+    ) -> i32;
+    pub fn b200nn_lm_generate_sampling(
+        m: *mut b200nn_lm,
+        prompt: *const u32,
+        prompt_len: usize,
+        max_new: usize,
+        top_k: usize,
+        temperature: f32,
+        rng_state: *mut u64,
+        out_tokens: *mut u32,
+        n_out: *mut usize,
+    ) -> i32;
+    pub fn b200nn_kvcache_acquire(c: *mut b200nn_kvcache, slot: *mut i32) -> i32;
+    pub fn b200nn_kvcache_release(c: *mut b200nn_kvcache, slot: i32) -> i32;
+    pub fn b200nn_kvcache_slot_len(c: *const b200nn_kvcache, slot: i32) -> usize;
+    pub fn b200nn_lm_step(
+        c: *mut b200nn_kvcache,
+        n_entries: usize,
+        slots: *const i32,
+        counts: *const usize,
+        tokens: *const u32,
+        n_want: usize,
+        want: *const usize,
+        logits: *mut f32,
     ) -> i32;
     pub fn b200nn_bpe_load(path: *const c_char, endoftext_id: u32, out: *mut *mut b200nn_bpe) -> i32;
     pub fn b200nn_bpe_create(

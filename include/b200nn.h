@@ -63,10 +63,11 @@ enum {
     B200NN_STOP_ON_EOS = 1u << 3,    /* stop before appending token 50256 (gpt2.rs:698-700)          */
     B200NN_TOKENS_ONLY = 1u << 4,    /* decode sessions: the step's logits are not written to memory (the greedy
                                         pick is taken in the LM head's epilogue); b200nn_session_logits fails */
-    B200NN_WEIGHTS_OUT_IN = 1u << 5  /* model creation: the four Linear weights of every block are given in Linear
+    B200NN_WEIGHTS_OUT_IN = 1u << 5, /* model creation: the four Linear weights of every block are given in Linear
                                         layout [out,in], as Gpt2Model::from_generic_weights holds them after the
                                         generic loader's Conv1D transposes (gpt2.rs:410-476, 1436-1500;
                                         model_generic.rs:222-277), instead of checkpoint layout [in,out] */
+    B200NN_LM_F32 = 1u << 6          /* b200nn_lm_create / _load: f32 weights, activations and arithmetic throughout */
 };
 
 typedef struct b200nn_ctx b200nn_ctx;
@@ -80,6 +81,7 @@ typedef struct b200nn_gpt2 b200nn_gpt2;
 typedef struct b200nn_kvcache b200nn_kvcache;
 typedef struct b200nn_session b200nn_session;
 typedef struct b200nn_block b200nn_block;
+typedef struct b200nn_lm b200nn_lm;
 
 /* ---- context: KernelRegistry::init_default (GH/nn/registry.rs:131-135) --------------------- */
 B200NN_API const char *b200nn_version(void);
@@ -131,6 +133,8 @@ B200NN_API int32_t b200nn_ctx_set_gemv_max_rows(b200nn_ctx *ctx, int32_t rows);
  * LayerNorm kernels inside the blocks: the residual GEMMs write fp16(x * scale) and per-tile row sums,
  * the q/k/v and MLP GEMMs normalise in their epilogue.  Measured slower than the kernels it removes
  * (the residual GEMMs then need complete sums, i.e. cluster splits); sessions read it when created.
+ * "lm_portion" (default 0 = 2048): most new tokens of one sequence a hybrid model's cache takes in a pass; a
+ * windowed layer's ring holds the window plus this many rows.  Read when a cache or session is created.
  * "persist" (default 0): decode steps of an int4 model run all transformer blocks as one cooperative
  * kernel (decode sessions whose shape it supports).  Measured slower than the per-op CUDA graph.
  * Its aids: "persist_min_rows" / "persist_max_rows" (batch range it is used for), "persist_prefetch_mb",
@@ -468,7 +472,7 @@ B200NN_API int32_t b200nn_session_logits(b200nn_session *s, float *out);
  * B200NN_PROF_COUNT entries. */
 enum {
     B200NN_PROF_EMBED = 0, B200NN_PROF_LAYERNORM, B200NN_PROF_LINEAR, B200NN_PROF_ATTENTION,
-    B200NN_PROF_LM_HEAD, B200NN_PROF_ARGMAX, B200NN_PROF_COUNT
+    B200NN_PROF_LM_HEAD, B200NN_PROF_ARGMAX, B200NN_PROF_RECURRENCE, B200NN_PROF_COUNT
 };
 B200NN_API int32_t b200nn_session_profile_step(b200nn_session *s, float *times_ms, uint64_t *linear_bytes);
 /* Device time of ONE kernel family in isolation: launches only that family's kernels of a decode
@@ -509,6 +513,44 @@ B200NN_API const char *b200nn_safetensors_last_error(void);
  * int4_group 0 builds the f32 model, otherwise the int4 model quantised with that group size. */
 B200NN_API int32_t b200nn_gpt2_load_safetensors(b200nn_ctx *ctx, const char *path, const b200nn_gpt2_config *cfg,
                                                 size_t int4_group, uint32_t flags, b200nn_gpt2 **out);
+
+/* ---- language models by architecture: registry, cache slots, serving step --------------------------
+ * b200nn_lm is a decoder-only model of any family: GPT-2 (a view of a b200nn_gpt2), or a hybrid decoder
+ * whose layers (gated delta rule or latent attention, each with an optional gated feed-forward) are listed in
+ * a config.json.  No counterpart in the reference, whose models are separate Rust types.
+ *   _create  config_json (the text) plus host f32 tensors by name
+ *   _load    a folder with config.json and model.safetensors (F32, F16 or BF16); the family follows from
+ *            the configuration's "architecture" ("Vivezen"), or its "architectures" / "model_type" (GPT-2)
+ * Default precision of hybrid models: bfloat16 weights and activations, f32 accumulation, norms, softmax,
+ * recurrence and residual; B200NN_LM_F32 selects f32 throughout (GPT-2 refuses it: B200NN_ERR_UNSUPPORTED). */
+typedef struct {
+    int32_t n_layer, width, vocab_size, n_positions /* 0: no limit of its own */, eos_token /* -1: none */;
+} b200nn_lm_info;
+B200NN_API int32_t b200nn_lm_create(b200nn_ctx *ctx, const char *config_json, size_t n_tensors, const char *const *names,
+                                    const float *const *data, const size_t *numels, uint32_t flags, b200nn_lm **out);
+B200NN_API int32_t b200nn_lm_load(b200nn_ctx *ctx, const char *dir, uint32_t flags, b200nn_lm **out);
+B200NN_API b200nn_lm *b200nn_gpt2_as_lm(b200nn_gpt2 *m); /* the same object: destroyed as the b200nn_gpt2 */
+B200NN_API void b200nn_lm_destroy(b200nn_lm *m);
+B200NN_API int32_t b200nn_lm_get_info(const b200nn_lm *m, b200nn_lm_info *out);
+B200NN_API const char *b200nn_lm_family(const b200nn_lm *m);
+/* Cache, decode session and generate loops over any family; see their GPT-2 forms for the arguments. */
+B200NN_API int32_t b200nn_lm_cache_create(b200nn_lm *m, size_t slots, size_t capacity, b200nn_kvcache **out);
+B200NN_API int32_t b200nn_lm_session_create(b200nn_lm *m, size_t batch, size_t capacity, uint32_t flags, b200nn_session **out);
+B200NN_API int32_t b200nn_lm_generate_batch(b200nn_lm *m, const uint32_t *prompts, size_t batch, size_t prompt_len,
+                                            size_t max_new, uint32_t flags, uint32_t *out_tokens, size_t *out_lens);
+B200NN_API int32_t b200nn_lm_generate_sampling(b200nn_lm *m, const uint32_t *prompt, size_t prompt_len, size_t max_new,
+                                               size_t top_k, float temperature, uint64_t *rng_state, uint32_t *out_tokens,
+                                               size_t *n_out);
+/* Requests of unequal length: each holds one slot of a cache from acquire to release (an empty sequence to
+ * begin with).  A step brings, for each of n_entries acquired slots, its next counts[i] tokens (tokens: all
+ * entries' one after the other), appends them to the slots' sequences and writes the logits [n_want, vocab]
+ * of the rows want[] (indices into tokens) to the host.  Portions may be cut anywhere; long ones run in
+ * several passes.  Synchronises. */
+B200NN_API int32_t b200nn_kvcache_acquire(b200nn_kvcache *c, int32_t *slot);
+B200NN_API int32_t b200nn_kvcache_release(b200nn_kvcache *c, int32_t slot);
+B200NN_API size_t b200nn_kvcache_slot_len(const b200nn_kvcache *c, int32_t slot);
+B200NN_API int32_t b200nn_lm_step(b200nn_kvcache *c, size_t n_entries, const int32_t *slots, const size_t *counts,
+                                  const uint32_t *tokens, size_t n_want, const size_t *want, float *logits);
 
 /* ---- Gpt2Tokenizer (crates/core/gpu-host/src/tokenizer.rs:34-62) ---------------------------------
  * Host code.  The reference wraps tiktoken-rs' r50k_base; here the byte-level BPE is implemented over a
