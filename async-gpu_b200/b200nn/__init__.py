@@ -67,6 +67,18 @@ class _LmInfo(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layer", "width", "vocab_size", "n_positions", "eos_token")]
 
 
+class _LatentShape(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "window")] + [("scale", C.c_float)]
+
+
+class _DeltaShape(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "conv")] + [("eps", C.c_float)]
+
+
+class _DeltaWeights(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("conv", "a_exp", "dt_bias", "norm")]
+
+
 class _Weights(C.Structure):
     _fields_ = [("wte", _f32p), ("wpe", _f32p), ("ln_f_weight", _f32p), ("ln_f_bias", _f32p),
                 ("layers", C.POINTER(_LayerW))]
@@ -193,6 +205,10 @@ def load_library() -> C.CDLL:
             "b200nn_kvcache_acquire": (i32, [vp, C.POINTER(i32)]), "b200nn_kvcache_release": (i32, [vp, i32]),
             "b200nn_kvcache_slot_len": (sz, [vp, i32]),
             "b200nn_lm_step": (i32, [vp, sz, C.POINTER(i32), szp, _u32p, sz, szp, _f32p]),
+            "b200nn_latent_prefill_attention": (i32, [vp, C.POINTER(_LatentShape), u32, vp, vp, vp, vp, i32, i32, i32, i32, vp, vp]),
+            "b200nn_latent_decode_attention": (i32, [vp, C.POINTER(_LatentShape), u32, vp, vp, vp, i32, vp, vp, i32, i32, vp]),
+            "b200nn_delta_rule": (i32, [vp, C.POINTER(_DeltaShape), u32, vp, C.POINTER(_DeltaWeights), vp, vp, vp, vp, i32, i32, i32,
+                                        vp, vp, vp]),
             "b200nn_bpe_load": (i32, [C.c_char_p, u32, vpp]),
             "b200nn_bpe_create": (i32, [C.c_char_p, szp, _u32p, sz, u32, vpp]),
             "b200nn_bpe_destroy": (None, [vp]), "b200nn_bpe_vocab_size": (sz, [vp]),

@@ -359,7 +359,7 @@ class DecodeSession:
         return out[:, : n.value]
 
     def logits(self):
-        out = np.empty((self.batch, self.model.config.vocab_size), dtype=np.float32)
+        out = np.empty((self.batch, self.model.vocab_size), dtype=np.float32)
         self.reg.check(self.reg.lib.b200nn_session_logits(self.h, out.ctypes.data_as(_f32p)))
         return out
 

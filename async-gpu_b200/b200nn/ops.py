@@ -6,7 +6,7 @@ import ctypes as C
 import numpy as np
 
 from . import (ACT_GELU_SIGMOID, ACT_GELU_TANH, ACT_RELU, ACT_SIGMOID, ACT_SILU, ERR_SHAPE, GpuTensor, KernelRegistry, NnError, _f32,
-               _f32p, _out, _u32p, load_library)
+               _f32p, _out, _u32p, _DeltaShape, _DeltaWeights, _LatentShape, load_library)
 
 
 # ---- quantize (ops/quantize.rs) ----
@@ -203,3 +203,24 @@ def decode_attention_f16(q_ptr, k_cache_ptr, v_cache_ptr, batch, n_heads, capaci
     """One query row per sequence against the first ``ctx_len`` cached positions, fp16 device buffers."""
     reg.check(reg.lib.b200nn_decode_attention_f16(reg.h, q_ptr, k_cache_ptr, v_cache_ptr, batch, n_heads, capacity,
                                                   ctx_len, out_ptr))
+
+
+def latent_prefill_attention(shape, q_ptr, kv_ptr, latent_ptr, gate_ptr, n_rows, k_rows, n_seq, max_n, seq_ptr, out_ptr, reg, flags=0):
+    """Windowed attention of prompt rows over expanded keys and values (device pointers as ints); ``shape`` is
+    (heads, dim, rot_dim, vdim, kv_rank, window, scale)."""
+    reg.check(reg.lib.b200nn_latent_prefill_attention(reg.h, C.byref(_LatentShape(*shape)), flags, q_ptr, kv_ptr, latent_ptr, gate_ptr,
+                                                      n_rows, k_rows, n_seq, max_n, seq_ptr, out_ptr))
+
+
+def latent_decode_attention(shape, q_ptr, qlat_ptr, cache_ptr, ring, pos_ptr, slot_ptr, n_rows, capacity, out_ptr, reg, flags=0):
+    """One query per row against cached latents."""
+    reg.check(reg.lib.b200nn_latent_decode_attention(reg.h, C.byref(_LatentShape(*shape)), flags, q_ptr, qlat_ptr, cache_ptr, ring, pos_ptr,
+                                                     slot_ptr, n_rows, capacity, out_ptr))
+
+
+def delta_rule(shape, weights, proj_ptr, conv_state_ptr, state_ptr, pos_ptr, slot_ptr, n_rows, out_ptr, reg, n_seq=0, max_n=0, seq_ptr=None,
+               scratch_ptr=None, flags=0):
+    """Gated delta rule; ``shape`` is (heads, kv_heads, dim, vdim, conv, eps), ``weights`` the device pointers
+    (conv, a_exp, dt_bias, norm).  ``n_seq`` 0: one token per row, else prompt portions."""
+    reg.check(reg.lib.b200nn_delta_rule(reg.h, C.byref(_DeltaShape(*shape)), flags, proj_ptr, C.byref(_DeltaWeights(*weights)), conv_state_ptr,
+                                        state_ptr, pos_ptr, slot_ptr, n_rows, n_seq, max_n, seq_ptr, scratch_ptr, out_ptr))

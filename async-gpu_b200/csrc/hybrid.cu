@@ -709,7 +709,7 @@ int b200nn_hybrid::latent_layer(Workspace &ws, b200nn_kvcache &kv, LayerState &s
             TRY(launch_grouped_f32(ctx, (const float *)lw.ukv_rows->p, 1, L.kv_w(), L.rank_p, (const float *)ws.lin->p, L.ld(), 0, sm.k_rows, e, 0));
         }
         prof_mark(ctx, p.prof, B200NN_PROF_LINEAR);
-        TRY(launch_latent_prefill(ctx, L, b16, ws.q->p, ws.kvx->p, ws.lin->p, sm, (const float *)ws.gate->p, ws.att->p));
+        TRY(launch_latent_prefill(ctx, L, b16, p.T, ws.q->p, ws.kvx->p, ws.lin->p, sm, (const float *)ws.gate->p, ws.att->p));
         prof_mark(ctx, p.prof, B200NN_PROF_ATTENTION);
     }
     TRY(resid_linear(lw.o, ws.att->p, p.T, (float *)ws.x->p));

@@ -35,8 +35,12 @@ int launch_rope_heads(b200nn_ctx *ctx, float *q, int n_rows, int heads, int head
 // Cache rows of each sequence's window keys -> lin [k_rows][ld].
 int launch_latent_gather(b200nn_ctx *ctx, const LatentDims &d, bool b16, const void *cache, int ring, const SeqMap &sm, void *lin);
 // Attention of prompt rows over expanded keys and values; out [row][head][vdim_p] times the gate.
-int launch_latent_prefill(b200nn_ctx *ctx, const LatentDims &d, bool b16, const void *q, const void *kvx, const void *lin,
+int launch_latent_prefill(b200nn_ctx *ctx, const LatentDims &d, bool b16, int n_rows, const void *q, const void *kvx, const void *lin,
                           const SeqMap &sm, const float *gate, void *out);
+// Its tensor-core form (latent_attention_tc.cu): bfloat16, dim and vdim up to 128, rot_dim up to 64.
+bool latent_prefill_tc_supported(const b200nn_ctx *ctx, const LatentDims &d);
+int launch_latent_prefill_tc(b200nn_ctx *ctx, const LatentDims &d, int n_rows, const __nv_bfloat16 *q, const __nv_bfloat16 *kvx,
+                             const __nv_bfloat16 *lin, const SeqMap &sm, const float *gate, __nv_bfloat16 *out);
 // One query row per sequence against the cached latents: qlat [row][head][rank_p] (the unrotated query through
 // the key up-projection), q for the rotated part; out [row][head][rank_p], the attention-weighted latents.
 int launch_latent_decode(b200nn_ctx *ctx, const LatentDims &d, bool b16, const void *q, const void *qlat, const void *cache, int ring,

@@ -245,8 +245,11 @@ int launch_latent_gather(b200nn_ctx *ctx, const LatentDims &d, bool b16, const v
     return B200NN_OK;
 }
 
-int launch_latent_prefill(b200nn_ctx *ctx, const LatentDims &d, bool b16, const void *q, const void *kvx, const void *lin,
+int launch_latent_prefill(b200nn_ctx *ctx, const LatentDims &d, bool b16, int n_rows, const void *q, const void *kvx, const void *lin,
                           const SeqMap &sm, const float *gate, void *out) {
+    if (b16 && latent_prefill_tc_supported(ctx, d))
+        return launch_latent_prefill_tc(ctx, d, n_rows, (const __nv_bfloat16 *)q, (const __nv_bfloat16 *)kvx, (const __nv_bfloat16 *)lin, sm, gate,
+                                        (__nv_bfloat16 *)out);
     if (d.vdim_p > 512) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "latent attention: vdim > 512");
     const dim3 grid(d.heads, sm.max_n, sm.n_seq);
     if (sm.max_n > 65535 || sm.n_seq > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "latent attention: more than 65535 rows or sequences");

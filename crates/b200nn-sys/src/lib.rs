@@ -98,6 +98,41 @@ pub struct b200nn_lm_info {
     pub eos_token: i32,
 }
 
+/// Sizes of latent attention (every size a multiple of 16; `window` 0: none).
+#[repr(C)]
+#[derive(Clone, Copy, Debug, PartialEq)]
+pub struct b200nn_latent_shape {
+    pub heads: i32,
+    pub dim: i32,
+    pub rot_dim: i32,
+    pub vdim: i32,
+    pub kv_rank: i32,
+    pub window: i32,
+    pub scale: f32,
+}
+
+/// Sizes of the gated delta rule.
+#[repr(C)]
+#[derive(Clone, Copy, Debug, PartialEq)]
+pub struct b200nn_delta_shape {
+    pub heads: i32,
+    pub kv_heads: i32,
+    pub dim: i32,
+    pub vdim: i32,
+    pub conv: i32,
+    pub eps: f32,
+}
+
+/// Device pointers of the delta rule's small weights.
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct b200nn_delta_weights {
+    pub conv: *const f32,
+    pub a_exp: *const f32,
+    pub dt_bias: *const f32,
+    pub norm: *const f32,
+}
+
 /// `TransformerLayerWeights` (model.rs:112-139): host f32, dense weights in Conv1D layout [in,out].
 #[repr(C)]
 #[derive(Clone, Copy)]
@@ -741,6 +776,52 @@ extern "C" {
         n_want: usize,
         want: *const usize,
         logits: *mut f32,
+    ) -> i32;
+    pub fn b200nn_latent_prefill_attention(
+        ctx: *mut b200nn_ctx,
+        shape: *const b200nn_latent_shape,
+        flags: u32,
+        q_dev: *const c_void,
+        kv_dev: *const c_void,
+        latent_dev: *const c_void,
+        gate_dev: *const f32,
+        n_rows: i32,
+        k_rows: i32,
+        n_seq: i32,
+        max_n: i32,
+        seq_dev: *const i32,
+        out_dev: *mut c_void,
+    ) -> i32;
+    pub fn b200nn_latent_decode_attention(
+        ctx: *mut b200nn_ctx,
+        shape: *const b200nn_latent_shape,
+        flags: u32,
+        q_dev: *const c_void,
+        qlat_dev: *const c_void,
+        cache_dev: *const c_void,
+        ring: i32,
+        pos_dev: *const i32,
+        slot_dev: *const i32,
+        n_rows: i32,
+        capacity: i32,
+        out_dev: *mut c_void,
+    ) -> i32;
+    pub fn b200nn_delta_rule(
+        ctx: *mut b200nn_ctx,
+        shape: *const b200nn_delta_shape,
+        flags: u32,
+        proj_dev: *const f32,
+        w: *const b200nn_delta_weights,
+        conv_state_dev: *mut f32,
+        state_dev: *mut f32,
+        pos_dev: *const i32,
+        slot_dev: *const i32,
+        n_rows: i32,
+        n_seq: i32,
+        max_n: i32,
+        seq_dev: *const i32,
+        scratch_dev: *mut f32,
+        out_dev: *mut c_void,
     ) -> i32;
     pub fn b200nn_bpe_load(path: *const c_char, endoftext_id: u32, out: *mut *mut b200nn_bpe) -> i32;
     pub fn b200nn_bpe_create(

@@ -552,6 +552,47 @@ B200NN_API size_t b200nn_kvcache_slot_len(const b200nn_kvcache *c, int32_t slot)
 B200NN_API int32_t b200nn_lm_step(b200nn_kvcache *c, size_t n_entries, const int32_t *slots, const size_t *counts,
                                   const uint32_t *tokens, size_t n_want, const size_t *want, float *logits);
 
+/* The hybrid decoder's sequence mechanisms as stream-ordered operations on caller-owned device buffers (the
+ * kernels the models launch).  16-bit buffers are bfloat16; with B200NN_LM_F32 in flags they are f32.  Every
+ * size is a multiple of 16, every buffer 16-byte aligned; index arrays are int32 on the device.
+ *
+ * Latent attention.  A cache row is [kv_rank latent | rot_dim rotated key part]; window 0 means none.
+ *   prefill: q [n_rows][heads][dim + rot_dim], kv [k_rows] x ([heads][dim] keys, [heads][vdim] values), latent
+ *     [k_rows] cache rows, gate f32 [n_rows][heads], out [n_rows][heads][vdim] times the gate.  seq [5][n_seq]:
+ *     first row, rows (the largest is max_n), past positions, first key row, position of the first key row.
+ *   decode: one query per row: qlat [n_rows][heads][kv_rank] (the unrotated query through the key
+ *     up-projection), q as above for its rotated part, cache [slots][ring] cache rows (position p in row
+ *     p % ring; ring a multiple of 128), pos and slot per row (slot NULL: slot = row); out
+ *     [n_rows][heads][kv_rank], the weighted latents.  capacity bounds the positions. */
+typedef struct {
+    int32_t heads, dim, rot_dim, vdim, kv_rank, window;
+    float scale;
+} b200nn_latent_shape;
+B200NN_API int32_t b200nn_latent_prefill_attention(b200nn_ctx *ctx, const b200nn_latent_shape *shape, uint32_t flags, const void *q_dev,
+                                                   const void *kv_dev, const void *latent_dev, const float *gate_dev, int32_t n_rows,
+                                                   int32_t k_rows, int32_t n_seq, int32_t max_n, const int32_t *seq_dev, void *out_dev);
+B200NN_API int32_t b200nn_latent_decode_attention(b200nn_ctx *ctx, const b200nn_latent_shape *shape, uint32_t flags, const void *q_dev,
+                                                  const void *qlat_dev, const void *cache_dev, int32_t ring, const int32_t *pos_dev,
+                                                  const int32_t *slot_dev, int32_t n_rows, int32_t capacity, void *out_dev);
+/* Gated delta rule with its short convolution, norms and output gate.  proj f32 [n_rows] x ([kv_heads][dim] q,
+ * [kv_heads][dim] k, [heads][vdim] v, [heads][vdim] gate, [heads] step-size and [heads] decay inputs); weights
+ * f32 on the device: conv [2 kv_heads dim + heads vdim][conv taps], a_exp [heads] = exp(A_log), dt_bias [heads],
+ * norm [vdim]; conv_state f32 [slots][taps][2 kv_heads dim + heads vdim], state f32 [slots][heads][dim][vdim];
+ * out [n_rows][heads][vdim].  n_seq 0: one token per row.  Else prompt portions: seq [4][n_seq] (slot, first row,
+ * rows, past) followed by the sequence index of every row, slot per row given, and scratch f32 of
+ * n_rows * (2 kv_heads dim + 2 heads vdim + 2 heads). */
+typedef struct {
+    int32_t heads, kv_heads, dim, vdim, conv;
+    float eps;
+} b200nn_delta_shape;
+typedef struct {
+    const float *conv, *a_exp, *dt_bias, *norm;
+} b200nn_delta_weights;
+B200NN_API int32_t b200nn_delta_rule(b200nn_ctx *ctx, const b200nn_delta_shape *shape, uint32_t flags, const float *proj_dev,
+                                     const b200nn_delta_weights *w, float *conv_state_dev, float *state_dev, const int32_t *pos_dev,
+                                     const int32_t *slot_dev, int32_t n_rows, int32_t n_seq, int32_t max_n, const int32_t *seq_dev,
+                                     float *scratch_dev, void *out_dev);
+
 /* ---- Gpt2Tokenizer (crates/core/gpu-host/src/tokenizer.rs:34-62) ---------------------------------
  * Host code.  The reference wraps tiktoken-rs' r50k_base; here the byte-level BPE is implemented over a
  * vocabulary given at run time: a file in tiktoken's format (one "base64(token bytes) rank" per
