@@ -206,7 +206,7 @@ def load_library() -> C.CDLL:
             "b200nn_kvcache_slot_len": (sz, [vp, i32]),
             "b200nn_lm_step": (i32, [vp, sz, C.POINTER(i32), szp, _u32p, sz, szp, _f32p]),
             "b200nn_latent_prefill_attention": (i32, [vp, C.POINTER(_LatentShape), u32, vp, vp, vp, vp, i32, i32, i32, i32, vp, vp]),
-            "b200nn_latent_decode_attention": (i32, [vp, C.POINTER(_LatentShape), u32, vp, vp, vp, i32, vp, vp, i32, i32, vp]),
+            "b200nn_latent_decode_attention": (i32, [vp, C.POINTER(_LatentShape), u32, vp, vp, vp, i32, vp, vp, i32, i32, i32, vp]),
             "b200nn_delta_rule": (i32, [vp, C.POINTER(_DeltaShape), u32, vp, C.POINTER(_DeltaWeights), vp, vp, vp, vp, i32, i32, i32,
                                         vp, vp, vp]),
             "b200nn_bpe_load": (i32, [C.c_char_p, u32, vpp]),

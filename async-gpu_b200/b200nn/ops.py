@@ -212,10 +212,10 @@ def latent_prefill_attention(shape, q_ptr, kv_ptr, latent_ptr, gate_ptr, n_rows,
                                                       n_rows, k_rows, n_seq, max_n, seq_ptr, out_ptr))
 
 
-def latent_decode_attention(shape, q_ptr, qlat_ptr, cache_ptr, ring, pos_ptr, slot_ptr, n_rows, capacity, out_ptr, reg, flags=0):
+def latent_decode_attention(shape, q_ptr, qlat_ptr, cache_ptr, ring, pos_ptr, slot_ptr, n_slots, n_rows, capacity, out_ptr, reg, flags=0):
     """One query per row against cached latents."""
     reg.check(reg.lib.b200nn_latent_decode_attention(reg.h, C.byref(_LatentShape(*shape)), flags, q_ptr, qlat_ptr, cache_ptr, ring, pos_ptr,
-                                                     slot_ptr, n_rows, capacity, out_ptr))
+                                                     slot_ptr, n_slots, n_rows, capacity, out_ptr))
 
 
 def delta_rule(shape, weights, proj_ptr, conv_state_ptr, state_ptr, pos_ptr, slot_ptr, n_rows, out_ptr, reg, n_seq=0, max_n=0, seq_ptr=None,

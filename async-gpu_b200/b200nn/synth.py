@@ -85,3 +85,63 @@ def int4_linear_case(seed: int, m: int, k: int, n: int, group: int = 128):
     scales = g.uniform(0.005, 0.02, size=(n_groups, n)).astype(np.float16).astype(np.float32)
     x = g.standard_normal((m, k), dtype=np.float32)
     return packed, scales, x, q
+
+
+def hybrid_config(width, layers, vocab, heads, kv_heads, dim, rot_dim, kv_rank, q_rank, window, ff, conv=4):
+    """config.json of a Vivezen decoder whose every fourth layer is latent attention and the others gated delta
+    rule, all with a feed-forward (head sizes equal for both mixers)."""
+    lat = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": ff},
+           "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": dim, "kv_rank": kv_rank, "q_rank": q_rank, "mask": {"size": window},
+                     "rot": {"base": 10000.0, "dims": rot_dim}, "scale": (dim + rot_dim) ** -0.5}}
+    dlt = {"type": "delta", "mlp": {"kind": "dense", "ff": ff},
+           "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": conv}}
+    return {"architecture": "Vivezen", "width": width, "vocab": vocab, "norm": {"eps": 1e-5},
+            "layers": [lat if i % 4 == 3 else dlt for i in range(layers)]}
+
+
+def hybrid_weights(cfg, base_seed=BASE_SEED):
+    """Random f32 weights of a hybrid decoder by tensor name: matrices with unit row gain, norms of one, decays spread
+    from a few tokens to hundreds."""
+    d, out = cfg["width"], {}
+
+    def mat(name, *shape):
+        out[name] = np.random.default_rng(base_seed + len(out)).standard_normal(shape, dtype=np.float32) * np.float32(shape[-1] ** -0.5)
+
+    def ones(name, n):
+        out[name] = np.ones(n, dtype=np.float32)
+
+    mat("embed", cfg["vocab"], d)
+    ones("final.norm", d)
+    for i, layer in enumerate(cfg["layers"]):
+        p, x = f"l{i}.", layer["mixer"]
+        m = p + "mix."
+        ones(p + "norm1", d)
+        if layer["type"] == "delta":
+            H, KH, dim, vd = x["heads"], x["kv_heads"], x["dim"], x["vdim"]
+            for n, c in (("q", KH * dim), ("k", KH * dim), ("v", H * vd)):
+                mat(m + n, c, d)
+                mat(m + n + ".conv", c, x["conv"])
+            for n, c in (("b", H), ("a", H), ("g", H * vd)):
+                mat(m + n, c, d)
+            out[m + "A_log"] = np.linspace(-4.0, 0.5, H, dtype=np.float32)
+            out[m + "dt_bias"] = np.full(H, -1.0, dtype=np.float32)
+            ones(m + "norm", vd)
+            mat(m + "o", d, H * vd)
+        else:
+            H, dim, rd, vd, R, Q = (x[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+            mat(m + "dq", Q, d)
+            ones(m + "dq.norm", Q)
+            mat(m + "uq", H * (dim + rd), Q)
+            mat(m + "dkv", R + rd, d)
+            ones(m + "dkv.norm", R)
+            mat(m + "uk", H * dim, R)
+            mat(m + "uv", H * vd, R)
+            mat(m + "g", H, d)
+            mat(m + "o", d, H * vd)
+        if layer.get("mlp"):
+            ff = layer["mlp"]["ff"]
+            ones(p + "norm2", d)
+            mat(p + "mlp.gate", ff, d)
+            mat(p + "mlp.up", ff, d)
+            mat(p + "mlp.down", d, ff)
+    return out

@@ -50,17 +50,17 @@ extern "C" int32_t b200nn_latent_prefill_attention(b200nn_ctx *ctx, const b200nn
 
 extern "C" int32_t b200nn_latent_decode_attention(b200nn_ctx *ctx, const b200nn_latent_shape *shape, uint32_t flags, const void *q_dev,
                                                   const void *qlat_dev, const void *cache_dev, int32_t ring, const int32_t *pos_dev,
-                                                  const int32_t *slot_dev, int32_t n_rows, int32_t capacity, void *out_dev) {
+                                                  const int32_t *slot_dev, int32_t n_slots, int32_t n_rows, int32_t capacity, void *out_dev) {
     LatentDims d;
-    if (!ctx || !shape || !pos_dev || n_rows <= 0 || ring <= 0 || capacity <= 0) return B200NN_ERR_ARG;
+    if (!ctx || !shape || !pos_dev || n_rows <= 0 || n_slots <= 0 || ring <= 0 || capacity <= 0) return B200NN_ERR_ARG;
     if (!latent_dims(shape, &d)) return set_error(ctx, B200NN_ERR_SHAPE, "latent attention: sizes must be positive multiples of 16");
     if (ring % 128 || (d.window ? ring < d.window : ring < capacity))
         return set_error(ctx, B200NN_ERR_SHAPE, "latent attention: the ring must be a multiple of 128 rows and hold the window");
     if (unaligned({q_dev, qlat_dev, cache_dev, out_dev})) return set_error(ctx, B200NN_ERR_ARG, "latent attention: buffers must be 16-byte aligned");
     CK(ctx, cudaSetDevice(ctx->device));
-    const size_t need = latent_decode_part_floats(ctx, d, n_rows, capacity) * sizeof(float);
+    const size_t need = latent_decode_part_floats(ctx, d, !(flags & B200NN_LM_F32), n_rows, capacity) * sizeof(float);
     if (need) TRY(ensure_scratch(ctx, need, 0));
-    return launch_latent_decode(ctx, d, !(flags & B200NN_LM_F32), q_dev, qlat_dev, cache_dev, ring, RowMap{pos_dev, 1, slot_dev}, n_rows, capacity,
+    return launch_latent_decode(ctx, d, !(flags & B200NN_LM_F32), q_dev, qlat_dev, cache_dev, ring, (size_t)n_slots * ring, RowMap{pos_dev, 1, slot_dev}, n_rows, capacity,
                                 out_dev, ctx->scratch);
 }
 

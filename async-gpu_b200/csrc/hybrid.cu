@@ -677,14 +677,14 @@ int b200nn_hybrid::latent_layer(Workspace &ws, b200nn_kvcache &kv, LayerState &s
     if (p.decode) {
         TRY(need(&ws.qlat, (size_t)p.T * H * L.rank_p * es));
         TRY(need(&ws.olat, (size_t)p.T * H * L.rank_p * es));
-        TRY(need(&ws.part, latent_decode_part_floats(ctx, L, p.T, (int)kv.cap) * 4));
+        TRY(need(&ws.part, latent_decode_part_floats(ctx, L, b16, p.T, (int)kv.cap) * 4));
         Epilogue e;
         e.out = ws.qlat->p;
         e.ldo = H * L.rank_p;
         e.out_half = act_type();
         TRY(run_grouped(lw.uk, ws.q->p, H * L.head_w(), p.T, e));
         prof_mark(ctx, p.prof, B200NN_PROF_LINEAR);
-        TRY(launch_latent_decode(ctx, L, b16, ws.q->p, ws.qlat->p, st.latent->p, st.ring, p.rows, p.T, (int)kv.cap, ws.olat->p,
+        TRY(launch_latent_decode(ctx, L, b16, ws.q->p, ws.qlat->p, st.latent->p, st.ring, kv.batch * st.ring, p.rows, p.T, (int)kv.cap, ws.olat->p,
                                  (float *)ws.part->p));
         prof_mark(ctx, p.prof, B200NN_PROF_ATTENTION);
         Epilogue v;

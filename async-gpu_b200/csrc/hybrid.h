@@ -43,9 +43,15 @@ int launch_latent_prefill_tc(b200nn_ctx *ctx, const LatentDims &d, int n_rows, c
                              const __nv_bfloat16 *lin, const SeqMap &sm, const float *gate, __nv_bfloat16 *out);
 // One query row per sequence against the cached latents: qlat [row][head][rank_p] (the unrotated query through
 // the key up-projection), q for the rotated part; out [row][head][rank_p], the attention-weighted latents.
+// cache_rows: all rows of the cache; cap bounds the positions; part: latent_decode_part_floats of scratch.
 int launch_latent_decode(b200nn_ctx *ctx, const LatentDims &d, bool b16, const void *q, const void *qlat, const void *cache, int ring,
-                         const RowMap &rows, int n_rows, int cap, void *out, float *part);
-size_t latent_decode_part_floats(const b200nn_ctx *ctx, const LatentDims &d, int n_rows, int cap);
+                         size_t cache_rows, const RowMap &rows, int n_rows, int cap, void *out, float *part);
+size_t latent_decode_part_floats(const b200nn_ctx *ctx, const LatentDims &d, bool b16, int n_rows, int cap);
+// Its tensor-core form (latent_decode_tc.cu): bfloat16, kv_rank up to 640, rot_dim up to 64.
+bool latent_decode_tc_supported(const b200nn_ctx *ctx, const LatentDims &d);
+size_t latent_decode_tc_part_floats(const b200nn_ctx *ctx, const LatentDims &d, int n_rows, int cap);
+int launch_latent_decode_tc(b200nn_ctx *ctx, const LatentDims &d, const __nv_bfloat16 *q, const __nv_bfloat16 *qlat, const __nv_bfloat16 *cache,
+                            int ring, size_t cache_rows, const RowMap &rows, int n_rows, int cap, __nv_bfloat16 *out, float *part);
 
 // ---- gated delta rule ------------------------------------------------------------------------------
 // Projection rows (f32): [q kv_heads*dim_p | k kv_heads*dim_p | v heads*vdim_p | gate heads*vdim_p | b heads |

@@ -267,12 +267,15 @@ int launch_latent_prefill(b200nn_ctx *ctx, const LatentDims &d, bool b16, int n_
     return B200NN_OK;
 }
 
-size_t latent_decode_part_floats(const b200nn_ctx *, const LatentDims &, int, int) { return 0; }
+size_t latent_decode_part_floats(const b200nn_ctx *ctx, const LatentDims &d, bool b16, int n_rows, int cap) {
+    return b16 && latent_decode_tc_supported(ctx, d) ? latent_decode_tc_part_floats(ctx, d, n_rows, cap) : 0;
+}
 
 int launch_latent_decode(b200nn_ctx *ctx, const LatentDims &d, bool b16, const void *q, const void *qlat, const void *cache, int ring,
-                         const RowMap &rows, int n_rows, int cap, void *out, float *part) {
-    (void)cap;
-    (void)part;
+                         size_t cache_rows, const RowMap &rows, int n_rows, int cap, void *out, float *part) {
+    if (b16 && latent_decode_tc_supported(ctx, d))
+        return launch_latent_decode_tc(ctx, d, (const __nv_bfloat16 *)q, (const __nv_bfloat16 *)qlat, (const __nv_bfloat16 *)cache, ring, cache_rows,
+                                       rows, n_rows, cap, (__nv_bfloat16 *)out, part);
     if (d.rank_p > 1024) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "latent attention: kv_rank > 1024");
     if (n_rows > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "latent attention: more than 65535 rows");
     const dim3 grid(d.heads, n_rows);

@@ -320,6 +320,175 @@ def attention_isolated(reg, hbm_peak, tf_peak, seqs=(256, 512, 1024), decode=Tru
     return out
 
 
+# --design vivezen: sizes of the hybrid decoder that resemble layers of real models, and the batches they run
+# name: (width, layers, vocab, heads, kv_heads, dim, rot_dim, kv_rank, q_rank, window, ff), sequences, prompt, decode steps
+HYBRID_SIZES = {
+    "w1024": ((1024, 8, 32000, 8, 4, 128, 64, 256, 512, 512, 2816), 64, 1024, 32),
+    "w2048": ((2048, 8, 32000, 16, 8, 128, 64, 512, 1024, 1024, 5632), 32, 2048, 32),
+    "w4096": ((4096, 4, 32000, 32, 16, 128, 64, 512, 1536, 1024, 11264), 16, 2048, 32),
+}
+
+
+def hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak):
+    """The hybrid decoder's sequence kernels alone, on device buffers, each between two CUDA events over a replayed
+    graph.  Prompt attention counts the visible (query, key) pairs only: 2 (dim + rot) + 2 vdim flops each and
+    head.  The recurrence counts 6 dim vdim flops per token and head (S^T k, S^T q, k u^T) against the f32 FMA
+    peak at the sampled clock (148 SMs x 128 lanes x 2 x 1.965 GHz = 74.4 TFLOP/s): state and everything
+    that enters it are f32.  Decode counts the window's cache rows (latent attention) or the state read and
+    written (delta rule); copies rotate through more than the L2."""
+    import torch
+    from b200nn import ops
+    width, layers, vocab, H, KH, dim, rot, rank, qr, window, ff = shape
+    stream = torch.cuda.ExternalStream(reg.stream)
+    dev = "cuda"
+    out = {}
+    f32_peak = 74.4
+    lat = (H, dim, rot, dim, rank, window, (dim + rot) ** -0.5)
+
+    def ints(*rows):
+        return torch.tensor([int(v) for r in rows for v in r], device=dev, dtype=torch.int32)
+
+    # latent attention, prompts
+    B = max(1, min(batch, 16384 // prompt))
+    T = B * prompt
+    q = torch.randn(T, H * (dim + rot), device=dev).to(torch.bfloat16)
+    kv = torch.randn(T, H * 2 * dim, device=dev).to(torch.bfloat16)
+    rows = torch.randn(T, rank + rot, device=dev).to(torch.bfloat16)
+    gate = torch.rand(T, H, device=dev)
+    o = torch.empty(T, H * dim, device=dev, dtype=torch.bfloat16)
+    r0 = [prompt * b for b in range(B)]
+    seq = ints(r0, [prompt] * B, [0] * B, r0, [0] * B)
+    call = lambda i: ops.latent_prefill_attention(lat, q.data_ptr(), kv.data_ptr(), rows.data_ptr(), gate.data_ptr(), T, T, B, prompt,
+                                                  seq.data_ptr(), o.data_ptr(), reg)
+    torch.cuda.synchronize()
+    call(0)
+    reg.synchronize()
+    us = _graph_time(reg, stream, call, 16)
+    pairs = sum(min(i + 1, window) for i in range(prompt)) * B * H
+    fl = pairs * 2 * (2 * dim + rot)
+    out["latent_prefill_tc_kernel"] = {"tokens": T, "us": round(us, 1), "tflops": round(fl / us / 1e6, 1), "frac_of_bf16_peak": round(fl / us / 1e6 / tf_peak, 4)}
+    del q, kv, rows, o
+    # latent attention, decoding with a full window
+    ring = -(-(window + 128) // 128) * 128
+    nbytes = batch * window * (rank + rot) * 2 + batch * H * (2 * rank + dim + rot) * 2
+    copies = max(2, int(300e6 // (batch * ring * (rank + rot) * 2)) + 1)
+    caches = [torch.randn(batch, ring, rank + rot, device=dev).to(torch.bfloat16) for _ in range(copies)]
+    q = torch.randn(batch, H * (dim + rot), device=dev).to(torch.bfloat16)
+    ql = torch.randn(batch, H * rank, device=dev).to(torch.bfloat16)
+    o = torch.empty_like(ql)
+    pos = ints([window + 5 + b % 100 for b in range(batch)])
+    call = lambda i: ops.latent_decode_attention(lat, q.data_ptr(), ql.data_ptr(), caches[i % copies].data_ptr(), ring, pos.data_ptr(), None, batch, batch,
+                                                 window + 128, o.data_ptr(), reg)
+    torch.cuda.synchronize()
+    call(0)
+    reg.synchronize()
+    us = _graph_time(reg, stream, call, 6 * copies)
+    out["latent_decode"] = {"rows": batch, "window": window, "us": round(us, 1), "GBps": round(nbytes / us / 1e3, 1),
+                            "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
+    del caches
+    # delta rule
+    sh = (H, KH, dim, dim, 4, 1e-5)
+    cw = 2 * KH * dim + H * dim
+    pw = cw + H * dim + 2 * H
+    wts = [torch.randn(cw, 4, device=dev), torch.full((H,), 0.1, device=dev), torch.zeros(H, device=dev), torch.ones(dim, device=dev)]
+    ptrs = tuple(t.data_ptr() for t in wts)
+    proj = torch.randn(max(T, batch), pw, device=dev)
+    conv = torch.zeros(batch, 4, cw, device=dev)
+    state = torch.zeros(batch, H, dim, dim, device=dev)
+    o = torch.empty(max(T, batch), H * dim, device=dev, dtype=torch.bfloat16)
+    scratch = torch.empty(T * (cw + 2 * H + H * dim), device=dev)
+    rpos, rslot = ints([i % prompt for i in range(T)]), ints([i // prompt for i in range(T)])
+    seq = ints(range(B), r0, [prompt] * B, [0] * B, [i // prompt for i in range(T)])
+    call = lambda i: ops.delta_rule(sh, ptrs, proj.data_ptr(), conv.data_ptr(), state.data_ptr(), rpos.data_ptr(), rslot.data_ptr(), T, o.data_ptr(),
+                                    reg, B, prompt, seq.data_ptr(), scratch.data_ptr())
+    torch.cuda.synchronize()
+    call(0)
+    reg.synchronize()
+    us = _graph_time(reg, stream, call, 6)
+    fl = 6 * dim * dim * H * T
+    out["delta_prompt"] = {"tokens": T, "sequences": B, "us": round(us, 1), "tflops_f32": round(fl / us / 1e6, 2),
+                           "frac_of_f32_peak": round(fl / us / 1e6 / f32_peak, 4)}
+    copies = max(2, int(300e6 // (state.numel() * 4)) + 1)
+    states = [torch.randn_like(state) * 0.01 for _ in range(copies)]
+    pos = ints([100] * batch)
+    call = lambda i: ops.delta_rule(sh, ptrs, proj.data_ptr(), conv.data_ptr(), states[i % copies].data_ptr(), pos.data_ptr(), None, batch, o.data_ptr(), reg)
+    torch.cuda.synchronize()
+    call(0)
+    reg.synchronize()
+    us = _graph_time(reg, stream, call, 6 * copies)
+    nbytes = 2 * state.numel() * 4 + batch * pw * 4 + batch * 4 * cw * 4 + batch * H * dim * 2
+    out["delta_step_kernel"] = {"rows": batch, "us": round(us, 1), "GBps": round(nbytes / us / 1e3, 1), "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
+    return out
+
+
+def run_design(args):
+    """Prefill and decode throughput of the hybrid decoder beside a GPT-2 of the same width, depth, vocabulary and
+    batch (f32 family: fp16 tensor-core operands), N = 1, state resident, device-timed; not the headline."""
+    import torch
+    import b200nn
+    from b200nn import DecodeSession, Gpt2Config, Gpt2Model, LanguageModel, synth
+    torch.cuda.set_device(0)
+    reg = b200nn.KernelRegistry(0)
+    for kv in args.tune:
+        key, val = kv.split("=")
+        reg.set_tuning(key, int(val))
+    stream = torch.cuda.ExternalStream(reg.stream)
+    hbm_peak, tf_peak, kind = peaks()
+    line = {"design": args.design, "peaks": {"hbm_GBps": hbm_peak, "bf16_tflops": tf_peak, "source": kind}, "data": "synthetic", "sizes": {}}
+
+    def timed(fn):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        with torch.cuda.stream(stream):
+            e0.record(stream)
+            fn()
+            e1.record(stream)
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1)
+
+    def measure(model, batch, prompt, steps, vocab):
+        ids = synth.token_ids(7, (batch, prompt), vocab)
+        s = DecodeSession(model, batch, prompt + 4 * steps + 8, flags=b200nn.TOKENS_ONLY)
+        s.prefill(ids)
+        pre = min(timed(lambda: s.prefill(ids)) for _ in range(2))
+        s.step(max(3, args.warmup))
+        dec = timed(lambda: s.step(steps))
+        fam, _ = s.profile_step()
+        return {"prefill_tokens_per_s": round(batch * prompt / pre * 1e3), "prefill_ms": round(pre, 2),
+                "decode_tokens_per_s": round(batch * steps / dec * 1e3), "decode_ms_per_step": round(dec / steps, 4),
+                "decode_family_ms_with_events": {k: round(v, 4) for k, v in fam.items()}}
+
+    sampler = ClockSampler(0)
+    sampler.start()
+    for name in (args.sizes.split(",") if args.sizes else HYBRID_SIZES):
+        shape, batch, prompt, steps = HYBRID_SIZES[name]
+        width, layers, vocab, H, KH, dim, rot, rank, qr, window, ff = shape
+        rec = {"config": dict(zip(("width", "layers", "vocab", "heads", "kv_heads", "dim", "rot_dim", "kv_rank", "q_rank", "window", "ff"), shape)),
+               "sequences": batch, "prompt": prompt, "kernels": hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak)}
+        if not args.kernels_only:
+            cfg = synth.hybrid_config(width, layers, vocab, H, KH, dim, rot, rank, qr, window, ff)
+            w = synth.hybrid_weights(cfg)
+            m = LanguageModel.from_weights(cfg, w, reg)
+            rec["parameters"] = sum(a.size for a in w.values())
+            del w
+            rec["vivezen_bf16"] = measure(m, batch, prompt, steps, vocab)
+            del m
+            reg.trim()
+            g = Gpt2Config(layers, width, width // 64, vocab, prompt + 4 * steps + 8)
+            gw = synth.gpt2_weights(g)
+            rec["gpt2_parameters"] = sum(a.size for a in gw.values())
+            m = Gpt2Model.from_weights(gw, g, reg)
+            del gw
+            rec["gpt2_f32_family"] = measure(m, batch, prompt, steps, vocab)
+            del m
+            reg.trim()
+        line["sizes"][name] = rec
+    if not args.kernels_only:
+        line["gpt2_attention"] = attention_isolated(reg, hbm_peak, tf_peak)
+    line["clocks"] = sampler.finish()
+    print(json.dumps(line), flush=True)
+    return 0
+
+
 def cpu_reference_form(steps=1):
     """The reference benchmark's first configuration the way the reference's CPU test runs it (tests_inference.rs:4393-4540): GPT-2
     Small, f32 weights, f64 accumulation, greedy decode WITHOUT a KV cache (every step recomputes the
@@ -603,7 +772,13 @@ def main():
     ap.add_argument("--cpu-steps", type=int, default=8)
     ap.add_argument("--cpu-prompt", type=int, default=32)
     ap.add_argument("--cpu-max-steps", type=int, default=64)
+    ap.add_argument("--design", default="", choices=["", "vivezen"],
+                    help="measure this model design at a few sizes beside a GPT-2 of equal width instead of the headline workload")
+    ap.add_argument("--sizes", default="", help="with --design: comma-separated subset of its sizes")
+    ap.add_argument("--kernels-only", action="store_true", help="with --design: only the isolated kernels")
     args = ap.parse_args()
+    if args.design:
+        return run_design(args)
     if args.impl == "reference":
         return run_reference(args)
     if args.isolated_only:

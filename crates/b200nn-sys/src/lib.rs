@@ -802,6 +802,7 @@ extern "C" {
         ring: i32,
         pos_dev: *const i32,
         slot_dev: *const i32,
+        n_slots: i32,
         n_rows: i32,
         capacity: i32,
         out_dev: *mut c_void,

@@ -561,7 +561,7 @@ B200NN_API int32_t b200nn_lm_step(b200nn_kvcache *c, size_t n_entries, const int
  *     [k_rows] cache rows, gate f32 [n_rows][heads], out [n_rows][heads][vdim] times the gate.  seq [5][n_seq]:
  *     first row, rows (the largest is max_n), past positions, first key row, position of the first key row.
  *   decode: one query per row: qlat [n_rows][heads][kv_rank] (the unrotated query through the key
- *     up-projection), q as above for its rotated part, cache [slots][ring] cache rows (position p in row
+ *     up-projection), q as above for its rotated part, cache [n_slots][ring] cache rows (position p in row
  *     p % ring; ring a multiple of 128), pos and slot per row (slot NULL: slot = row); out
  *     [n_rows][heads][kv_rank], the weighted latents.  capacity bounds the positions. */
 typedef struct {
@@ -573,7 +573,8 @@ B200NN_API int32_t b200nn_latent_prefill_attention(b200nn_ctx *ctx, const b200nn
                                                    int32_t k_rows, int32_t n_seq, int32_t max_n, const int32_t *seq_dev, void *out_dev);
 B200NN_API int32_t b200nn_latent_decode_attention(b200nn_ctx *ctx, const b200nn_latent_shape *shape, uint32_t flags, const void *q_dev,
                                                   const void *qlat_dev, const void *cache_dev, int32_t ring, const int32_t *pos_dev,
-                                                  const int32_t *slot_dev, int32_t n_rows, int32_t capacity, void *out_dev);
+                                                  const int32_t *slot_dev, int32_t n_slots, int32_t n_rows, int32_t capacity,
+                                                  void *out_dev);
 /* Gated delta rule with its short convolution, norms and output gate.  proj f32 [n_rows] x ([kv_heads][dim] q,
  * [kv_heads][dim] k, [heads][vdim] v, [heads][vdim] gate, [heads] step-size and [heads] decay inputs); weights
  * f32 on the device: conv [2 kv_heads dim + heads vdim][conv taps], a_exp [heads] = exp(A_log), dt_bias [heads],

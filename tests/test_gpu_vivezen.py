@@ -96,7 +96,7 @@ def check(got, want, tol, what=""):
     got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
     err = np.sqrt(((got - want) ** 2).mean(-1) / (want ** 2).mean())
     assert got.shape == want.shape and np.isfinite(got).all() and err.max() < tol, f"{what}: row {int(err.argmax())}, error {err.max():.2e}"
-    assert tol != TOL["bfloat16"] or len(err) < 8 or err.mean() < 0.025, f"{what}: mean error {err.mean():.2e}"
+    assert tol != TOL["bfloat16"] or err.size < 8 or err.mean() < 0.025, f"{what}: mean error {err.mean():.2e}"
 
 
 def run(rb, name, toks, portions):
@@ -380,7 +380,7 @@ def test_latent_decode_attention(reg, shape, spike, dtype):
     tp, ts = _ints(poss), _ints(slots)
     torch.cuda.synchronize()
     ops.latent_decode_attention((H, dim, rot, vdim, rank, window, scale), tq.data_ptr(), tql.data_ptr(), tc.data_ptr(), ring, tp.data_ptr(),
-                                ts.data_ptr(), B, cap, out.data_ptr(), reg, flags=0 if dtype == "bfloat16" else b200nn.LM_F32)
+                                ts.data_ptr(), B + 2, B, cap, out.data_ptr(), reg, flags=0 if dtype == "bfloat16" else b200nn.LM_F32)
     reg.synchronize()
     got = out.float().cpu().numpy()
     for b, p in enumerate(poss):
