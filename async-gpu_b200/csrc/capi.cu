@@ -111,6 +111,7 @@ extern "C" int32_t b200nn_ctx_set_tuning(b200nn_ctx *ctx, const char *key, int32
         if (ctx->trace) cudaMemset(ctx->trace, 0, 256 * sizeof(long long));
         if (!value && ctx->trace) { cudaFree(ctx->trace); ctx->trace = nullptr; }
     }
+    else if (!strcmp(key, "delta_cols")) ctx->delta_cols = value == 1 || value == 2 ? value : 0;
     else if (!strcmp(key, "lm_portion")) ctx->lm_portion = value < 0 ? 0 : value;
     else if (!strcmp(key, "gemv_max_rows")) ctx->gemv_max_rows = value < 0 ? 2 : value;
     else if (!strcmp(key, "fused_argmax")) ctx->fused_argmax = value ? 1 : 0;

@@ -86,5 +86,5 @@ extern "C" int32_t b200nn_delta_rule(b200nn_ctx *ctx, const b200nn_delta_shape *
     sm.n = seq_dev + 2 * n_seq;
     sm.past = seq_dev + 3 * n_seq;
     return launch_delta_prompt(ctx, d, b16, proj_dev, d.proj_w(), dw, conv_state_dev, state_dev, rows, sm, n_rows, seq_dev + 4 * n_seq, scratch_dev,
-                               scratch_dev + (size_t)n_rows * (d.conv_w() + 2 * d.heads), out_dev);
+                               scratch_dev + (size_t)n_rows * d.conv_ld(), out_dev);
 }

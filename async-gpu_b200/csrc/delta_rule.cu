@@ -4,8 +4,8 @@
 // state and one reduction instead of two.  Everything here is f32.
 //
 //   delta_step_kernel     decoding: convolution, norms, recurrence, output norm and gate of one token
-//   delta_conv_kernel     prompts: convolution + silu, unit norms, decay and step size of every row
-//   delta_scan_kernel     prompts: the recurrence (state columns are independent: a block owns 16 of them)
+//   delta_conv_kernel     prompts: convolution + silu, unit norms, k . q, decay and step size of every row
+//   delta_scan_kernel     prompts: the recurrence (state columns are independent: a block owns some of them)
 //   delta_out_kernel      prompts: output norm and gate
 //
 // The convolution's inputs are kept in a ring of `taps` rows per slot (position p in row p % taps): a token
@@ -57,10 +57,10 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         const int ch = which == 0 ? d.q_at() + kh * d.dim_p + t
                                   : which == 1 ? d.k_at() + kh * d.dim_p + (t - d.dim_p) : d.v_at() + h * d.vdim_p + (t - 2 * d.dim_p);
         const float x = p[ch];
-        const float *cwt = w.conv + (size_t)ch * d.taps;
-        float a = x * cwt[d.taps - 1];
+        const float *cwt = w.conv + ch;
+        float a = x * cwt[(size_t)(d.taps - 1) * cw];
         for (int j = 1; j < d.taps; ++j)
-            if (pos - j >= 0) a = fmaf(cring[(size_t)((pos - j) % d.taps) * cw + ch], cwt[d.taps - 1 - j], a);
+            if (pos - j >= 0) a = fmaf(cring[(size_t)((pos - j) % d.taps) * cw + ch], cwt[(size_t)(d.taps - 1 - j) * cw], a);
         if (which == 2 || h % group == 0) cring[(size_t)(pos % d.taps) * cw + ch] = x;
         sh[t] = silu_f(a); // q, k and v lie behind one another
     }
@@ -131,130 +131,275 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
 }
 
 // ---- prompts -----------------------------------------------------------------------------------------
-// Block = row; a warp takes one head of q, k or v at a time.
+// Columns of the convolved rows: q (scaled), k, v as in the projection, then per head the decay and the step size,
+// then per query/key head k . q; rows DeltaDims::conv_ld() apart.
+//
+// A warp takes four rows of one unit: a query/key head (both of its vectors) or a value head.  The eight warps of a
+// block take neighbouring rows, which share their convolution inputs in L1.
+constexpr int CONV_ROWS = 4;
 __global__ void __launch_bounds__(256)
 delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWeights w, const float *__restrict__ conv_state, RowMap rows,
-                  SeqMap sm, const int *__restrict__ row_seq, float *__restrict__ conv) {
+                  SeqMap sm, const int *__restrict__ row_seq, int n_rows, float *__restrict__ conv) {
     pdl_trigger();
     pdl_wait();
-    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int pos = row_pos(rows, row), slot = row_slot(rows, row), i = row - sm.row0[row_seq[row]], cw = d.conv_w();
-    const float *cring = conv_state + (size_t)slot * d.taps * cw;
-    float *o = conv + (size_t)row * (cw + 2 * d.heads);
-    const int units = 2 * d.kv_heads + d.heads;
-    for (int u = warp; u < units; u += 8) {
-        const bool isv = u >= 2 * d.kv_heads;
-        const int at = isv ? d.v_at() + (u - 2 * d.kv_heads) * d.vdim_p : u * d.dim_p, n = isv ? d.vdim_p : d.dim_p;
-        float s = 0.0f;
-        for (int j = lane; j < n; j += 32) {
-            const int ch = at + j;
-            const float *cwt = w.conv + (size_t)ch * d.taps;
-            float a = proj[(size_t)row * ldp + ch] * cwt[d.taps - 1];
-            for (int t = 1; t < d.taps; ++t) {
-                if (pos - t < 0) break;
-                const float x = i - t >= 0 ? proj[(size_t)(row - t) * ldp + ch] : cring[(size_t)((pos - t) % d.taps) * cw + ch];
-                a = fmaf(x, cwt[d.taps - 1 - t], a);
-            }
-            a = silu_f(a);
-            o[ch] = a;
-            s = fmaf(a, a, s);
-        }
-        if (!isv) {
-            s = warp_sum(s);
-            float f = 1.0f / sqrtf(s + 1e-6f);
-            if (u < d.kv_heads) f *= 1.0f / sqrtf((float)d.dim);
-            for (int j = lane; j < n; j += 32) o[at + j] *= f; // the lane's own values
-        }
+    const int r_first = (blockIdx.y * 8 + (threadIdx.x >> 5)) * CONV_ROWS, u = blockIdx.x, lane = threadIdx.x & 31;
+    const int cw = d.conv_w(), ld = d.conv_ld();
+    int pos[CONV_ROWS], back[CONV_ROWS]; // position; rows of the same sequence before it in the pass
+    const float *cring[CONV_ROWS];
+#pragma unroll
+    for (int r = 0; r < CONV_ROWS; ++r) {
+        const int row = min(r_first + r, n_rows - 1);
+        pos[r] = row_pos(rows, row);
+        back[r] = row - sm.row0[row_seq[row]];
+        cring[r] = conv_state + (size_t)row_slot(rows, row) * d.taps * cw;
     }
-    const float *p = proj + (size_t)row * ldp;
-    for (int h = threadIdx.x; h < d.heads; h += 256) {
-        o[cw + h] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
-        o[cw + d.heads + h] = sigmoid_f(p[d.b_at() + h]);
+    // channels ch .. ch+3 of row r_first + r after convolution and silu
+    auto channels = [&](int r, int ch) {
+        const float *p = proj + (size_t)min(r_first + r, n_rows - 1) * ldp;
+        const float4 x = *reinterpret_cast<const float4 *>(p + ch), w0 = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1) * cw + ch));
+        float4 a = make_float4(x.x * w0.x, x.y * w0.y, x.z * w0.z, x.w * w0.w);
+        for (int t = 1; t < d.taps && pos[r] - t >= 0; ++t) {
+            const float4 y = *reinterpret_cast<const float4 *>(back[r] >= t ? p - (size_t)t * ldp + ch : cring[r] + (size_t)((pos[r] - t) % d.taps) * cw + ch);
+            const float4 wt = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1 - t) * cw + ch));
+            a.x = fmaf(y.x, wt.x, a.x); a.y = fmaf(y.y, wt.y, a.y); a.z = fmaf(y.z, wt.z, a.z); a.w = fmaf(y.w, wt.w, a.w);
+        }
+        return make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
+    };
+    if (u >= d.kv_heads) { // a value head
+        const int h = u - d.kv_heads;
+        for (int j = lane * 4; j < d.vdim_p; j += 128) {
+            float4 v[CONV_ROWS];
+#pragma unroll
+            for (int r = 0; r < CONV_ROWS; ++r) v[r] = channels(r, d.v_at() + h * d.vdim_p + j);
+#pragma unroll
+            for (int r = 0; r < CONV_ROWS; ++r)
+                if (r_first + r < n_rows) *reinterpret_cast<float4 *>(conv + (size_t)(r_first + r) * ld + d.v_at() + h * d.vdim_p + j) = v[r];
+        }
+        if (lane < CONV_ROWS && r_first + lane < n_rows) {
+            const float *p = proj + (size_t)(r_first + lane) * ldp;
+            float *o = conv + (size_t)(r_first + lane) * ld;
+            o[d.decay_at() + h] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
+            o[d.beta_at() + h] = sigmoid_f(p[d.b_at() + h]);
+        }
+        return;
+    }
+    const float q_scale = 1.0f / sqrtf((float)d.dim);
+#pragma unroll
+    for (int half = 0; half < 2; ++half) { // two rows at a time
+        float4 q[2][2], k[2][2]; // [row][chunk of 128]; dim <= 256
+        float qq[2], kk[2], kq[2];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            qq[r] = kk[r] = kq[r] = 0.0f;
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const int j = lane * 4 + 128 * c;
+                float4 &a = q[r][c], &b = k[r][c];
+                a = b = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (j < d.dim_p) {
+                    a = channels(2 * half + r, d.q_at() + u * d.dim_p + j);
+                    b = channels(2 * half + r, d.k_at() + u * d.dim_p + j);
+                }
+                qq[r] += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
+                kk[r] += (b.x * b.x + b.y * b.y) + (b.z * b.z + b.w * b.w);
+                kq[r] += (a.x * b.x + a.y * b.y) + (a.z * b.z + a.w * b.w);
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int row = r_first + 2 * half + r;
+            const float fq = q_scale / sqrtf(warp_sum(qq[r]) + 1e-6f), fk = 1.0f / sqrtf(warp_sum(kk[r]) + 1e-6f);
+            const float dot = warp_sum(kq[r]) * fq * fk;
+            if (row >= n_rows) continue;
+            float *o = conv + (size_t)row * ld;
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                const int j = lane * 4 + 128 * c;
+                if (j < d.dim_p) {
+                    const float4 a = q[r][c], b = k[r][c];
+                    *reinterpret_cast<float4 *>(o + d.q_at() + u * d.dim_p + j) = make_float4(a.x * fq, a.y * fq, a.z * fq, a.w * fq);
+                    *reinterpret_cast<float4 *>(o + d.k_at() + u * d.dim_p + j) = make_float4(b.x * fk, b.y * fk, b.z * fk, b.w * fk);
+                }
+            }
+            if (lane == 0) o[d.kq_at() + u] = dot;
+        }
     }
 }
 
-// Block = (16 state columns, head, sequence), four warps of four columns; the eight lanes of a column hold its
-// dim entries 4 l + 32 m .. + 3.  Tokens come through shared memory CH at a time.  Also leaves the
-// convolution's last inputs in the cache (blocks of column group 0).
-template <int DM>
+// Pairs of f32 in one register pair: one instruction for two multiply-adds.
+__device__ __forceinline__ uint64_t f32x2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 f32x2_parts(uint64_t v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ void cp_async16(void *smem, const void *gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void *smem, const void *gmem) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+
+// Block = (16 NC state columns, head, sequence), four warps.  The eight lanes of a column group hold its dim entries
+// 4 l + 32 m .. + 3 of NC columns each (f32 pairs along dim).  Tokens come through shared memory CH at a time, the next
+// CH being copied under the current ones.  The state is held divided by the decay G accumulated since it was last
+// rescaled (S = G s), so that a token costs three multiply-adds per entry; it is rescaled when G falls below 2^-20.
+// Per token: both products against the old state, one reduction over the eight lanes (transposing: 2 NC values in
+// log steps), the write.  Also leaves the convolution's last inputs in the cache (blocks of column group 0).
+template <int DM, int NC>
 __global__ void __launch_bounds__(128)
 delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ conv, float *__restrict__ conv_state,
                   float *__restrict__ state, SeqMap sm, float *__restrict__ heads_out) {
-    constexpr int CH = DM <= 4 ? 32 : 16, DP = DM * 32;
-    __shared__ __align__(16) float sk[CH][DP], sq[CH][DP];
-    __shared__ float sv[CH][16], sg[CH], sb[CH], skq[CH];
+    constexpr int CH = DM <= 4 ? 16 : 8, DP = DM * 32, CB = 16 * NC;
+    struct Stage {
+        float k[CH][DP], q[CH][DP], v[CH][CB], s[CH][4]; // s: decay, step size, k . q
+    };
+    extern __shared__ __align__(16) uint8_t smem_raw[];
+    Stage *stages = reinterpret_cast<Stage *>(smem_raw);
     pdl_trigger();
     const int cg = blockIdx.x, h = blockIdx.y, sidx = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int cl = warp * 4 + (lane >> 3), part = lane & 7, col = cg * 16 + cl;
+    const int part = lane & 7, cl = (warp * 4 + (lane >> 3)) * NC, col = cg * CB + cl; // NC columns from col on
+    for (int i = tid; i < (int)(2 * sizeof(Stage) / 4); i += 128) reinterpret_cast<float *>(smem_raw)[i] = 0.0f; // entries past dim stay zero
     pdl_wait();
     const int n = sm.n[sidx], past = sm.past[sidx], slot = sm.slot[sidx], row0 = sm.row0[sidx];
-    const int group = d.heads / d.kv_heads, kh = h / group, cw = d.conv_w(), ldc = cw + 2 * d.heads;
+    const int group = d.heads / d.kv_heads, kh = h / group, cw = d.conv_w(), ldc = d.conv_ld();
     float *S = state + ((size_t)slot * d.heads + h) * d.dim_p * d.vdim_p + col;
-    float s[DM * 4];
+    uint64_t s[NC][DM * 2];
 #pragma unroll
     for (int m = 0; m < DM; ++m)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
+        for (int e = 0; e < 4; e += 2) {
             const int i = 32 * m + 4 * part + e;
-            s[4 * m + e] = i < d.dim_p && past > 0 ? S[(size_t)i * d.vdim_p] : 0.0f;
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                const bool in = i < d.dim_p && past > 0 && col + c < d.vdim_p;
+                s[c][2 * m + e / 2] = in ? f32x2(S[(size_t)i * d.vdim_p + c], S[(size_t)(i + 1) * d.vdim_p + c]) : 0ull;
+            }
         }
-    for (int t0 = 0; t0 < n; t0 += CH) {
+    auto copy = [&](int t0, Stage &st) {
+        const int nt = min(CH, n - t0), dv = d.dim_p >> 2, cv = min(CB, d.vdim_p - cg * CB) >> 2;
+        const float *c = conv + (size_t)(row0 + t0) * ldc;
+        for (int t = warp; t < nt; t += 4) { // a warp per token
+            const float *ct = c + (size_t)t * ldc;
+            for (int j = lane; j < dv; j += 32) {
+                cp_async16(&st.q[t][4 * j], ct + d.q_at() + kh * d.dim_p + 4 * j);
+                cp_async16(&st.k[t][4 * j], ct + d.k_at() + kh * d.dim_p + 4 * j);
+            }
+            if (lane < cv) cp_async16(&st.v[t][4 * lane], ct + d.v_at() + h * d.vdim_p + cg * CB + 4 * lane);
+            if (lane >= 29) {
+                const int j = lane - 29;
+                cp_async4(&st.s[t][j], ct + (j == 0 ? d.decay_at() + h : j == 1 ? d.beta_at() + h : d.kq_at() + kh));
+            }
+        }
+    };
+    __syncthreads();
+    copy(0, stages[0]);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    float G = 1.0f;
+    auto rescale = [&](float f) {
+        const uint64_t f2 = f32x2(f, f);
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int m = 0; m < DM * 2; ++m) s[c][m] = mul2(f2, s[c][m]);
+    };
+    for (int t0 = 0, b = 0; t0 < n; t0 += CH, b ^= 1) {
+        if (t0 + CH < n) copy(t0 + CH, stages[b ^ 1]);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const Stage &st = stages[b];
         const int nt = min(CH, n - t0);
-        __syncthreads();
-        for (int i = tid; i < nt * DP; i += 128) {
-            const int t = i / DP, j = i - t * DP;
-            const float *c = conv + (size_t)(row0 + t0 + t) * ldc;
-            sq[t][j] = j < d.dim_p ? c[d.q_at() + kh * d.dim_p + j] : 0.0f;
-            sk[t][j] = j < d.dim_p ? c[d.k_at() + kh * d.dim_p + j] : 0.0f;
-        }
-        for (int i = tid; i < nt * 16; i += 128)
-            sv[i >> 4][i & 15] = conv[(size_t)(row0 + t0 + (i >> 4)) * ldc + d.v_at() + h * d.vdim_p + cg * 16 + (i & 15)];
-        if (tid < nt) {
-            sg[tid] = conv[(size_t)(row0 + t0 + tid) * ldc + cw + h];
-            sb[tid] = conv[(size_t)(row0 + t0 + tid) * ldc + cw + d.heads + h];
-        }
-        __syncthreads();
-        for (int t = warp; t < nt; t += 4) {
-            float a = 0.0f;
-            for (int j = lane; j < DP; j += 32) a = fmaf(sk[t][j], sq[t][j], a);
-            a = warp_sum(a);
-            if (lane == 0) skq[t] = a;
-        }
-        __syncthreads();
         for (int t = 0; t < nt; ++t) {
-            float4 k[DM];
-            float ak = 0.0f, aq = 0.0f;
-#pragma unroll
-            for (int m = 0; m < DM; ++m) {
-                k[m] = *reinterpret_cast<const float4 *>(&sk[t][32 * m + 4 * part]);
-                const float4 q = *reinterpret_cast<const float4 *>(&sq[t][32 * m + 4 * part]);
-                ak = fmaf(s[4 * m], k[m].x, ak); ak = fmaf(s[4 * m + 1], k[m].y, ak);
-                ak = fmaf(s[4 * m + 2], k[m].z, ak); ak = fmaf(s[4 * m + 3], k[m].w, ak);
-                aq = fmaf(s[4 * m], q.x, aq); aq = fmaf(s[4 * m + 1], q.y, aq);
-                aq = fmaf(s[4 * m + 2], q.z, aq); aq = fmaf(s[4 * m + 3], q.w, aq);
+            const float4 sc = *reinterpret_cast<const float4 *>(st.s[t]);
+            G *= sc.x;
+            if (G < 9.5367431640625e-7f) { // the same in every thread of the block
+                rescale(G);
+                G = 1.0f;
             }
+            uint64_t k[DM * 2];
+            float r[2 * NC]; // s^T k of the NC columns, then s^T q
+            {
+                uint64_t ak[NC], aq[NC];
 #pragma unroll
-            for (int o = 1; o < 8; o <<= 1) {
-                ak += __shfl_xor_sync(0xffffffffu, ak, o);
-                aq += __shfl_xor_sync(0xffffffffu, aq, o);
-            }
-            const float g = sg[t], u = sb[t] * (sv[t][cl] - g * ak);
+                for (int c = 0; c < NC; ++c) ak[c] = aq[c] = 0ull;
 #pragma unroll
-            for (int m = 0; m < DM; ++m) {
-                s[4 * m] = fmaf(k[m].x, u, g * s[4 * m]);
-                s[4 * m + 1] = fmaf(k[m].y, u, g * s[4 * m + 1]);
-                s[4 * m + 2] = fmaf(k[m].z, u, g * s[4 * m + 2]);
-                s[4 * m + 3] = fmaf(k[m].w, u, g * s[4 * m + 3]);
+                for (int m = 0; m < DM; ++m) {
+                    const ulonglong2 kk = *reinterpret_cast<const ulonglong2 *>(&st.k[t][32 * m + 4 * part]);
+                    const ulonglong2 qq = *reinterpret_cast<const ulonglong2 *>(&st.q[t][32 * m + 4 * part]);
+                    k[2 * m] = kk.x;
+                    k[2 * m + 1] = kk.y;
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        ak[c] = fma2(s[c][2 * m], kk.x, ak[c]);
+                        aq[c] = fma2(s[c][2 * m], qq.x, aq[c]);
+                        ak[c] = fma2(s[c][2 * m + 1], kk.y, ak[c]);
+                        aq[c] = fma2(s[c][2 * m + 1], qq.y, aq[c]);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const float2 a = f32x2_parts(ak[c]), q = f32x2_parts(aq[c]);
+                    r[c] = a.x + a.y;
+                    r[NC + c] = q.x + q.y;
+                }
             }
-            if (part == 0) heads_out[((size_t)(row0 + t0 + t) * d.heads + h) * d.vdim_p + col] = fmaf(skq[t], u, g * aq);
+            // reduction over the eight lanes of the group: halve the values while there are several, then plain
+            int o = 4;
+#pragma unroll
+            for (int w = NC; w >= 1; w >>= 1, o >>= 1) {
+                const bool up = (lane & o) != 0;
+#pragma unroll
+                for (int i = 0; i < w; ++i) {
+                    const float send = up ? r[i] : r[i + w], keep = up ? r[i + w] : r[i];
+                    r[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            }
+            for (; o; o >>= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], o);
+            // lanes with bit 4 clear now hold s^T k, the others s^T q, of column idx
+            const int idx = NC == 1 ? 0 : (lane >> 1) & 1;
+            const float mine = G * r[0], other = __shfl_xor_sync(0xffffffffu, mine, 4);
+            const float u_own = sc.y * (st.v[t][cl + idx] - ((lane & 4) ? other : mine));
+            if ((lane & 4) && !(lane & 1) && (NC == 2 || !(lane & 2)) && col + idx < d.vdim_p)
+                heads_out[((size_t)(row0 + t0 + t) * d.heads + h) * d.vdim_p + col + idx] = fmaf(sc.z, u_own, mine);
+            const float us = __fdividef(u_own, G);
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                const float u = NC == 1 ? us : __shfl_sync(0xffffffffu, us, (lane & 24) | (c << 1));
+                const uint64_t u2 = f32x2(u, u);
+#pragma unroll
+                for (int m = 0; m < DM * 2; ++m) s[c][m] = fma2(k[m], u2, s[c][m]);
+            }
         }
+        __syncthreads();
     }
+    rescale(G);
 #pragma unroll
     for (int m = 0; m < DM; ++m)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
+        for (int e = 0; e < 4; e += 2) {
             const int i = 32 * m + 4 * part + e;
-            if (i < d.dim_p) S[(size_t)i * d.vdim_p] = s[4 * m + e];
+#pragma unroll
+            for (int c = 0; c < NC; ++c)
+                if (i < d.dim_p && col + c < d.vdim_p) {
+                    const float2 v = f32x2_parts(s[c][2 * m + e / 2]);
+                    S[(size_t)i * d.vdim_p + c] = v.x;
+                    S[(size_t)(i + 1) * d.vdim_p + c] = v.y;
+                }
         }
     if (cg == 0) {
         float *cring = conv_state + (size_t)slot * d.taps * cw;
@@ -281,13 +426,28 @@ delta_out_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const flo
     const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (unit >= n_rows * d.heads) return;
     const int row = unit / d.heads, h = unit - row * d.heads;
-    const float *o = heads_out + (size_t)unit * d.vdim_p;
+    const float *o = heads_out + (size_t)unit * d.vdim_p, *g = proj + (size_t)row * ldp + d.g_at() + h * d.vdim_p;
+    float4 v[2]; // the first 256 columns stay in registers
     float s = 0.0f;
-    for (int j = lane; j < d.vdim; j += 32) s = fmaf(o[j], o[j], s);
-    s = warp_sum(s);
-    const float rn = 1.0f / sqrtf(s / (float)d.vdim + d.eps);
-    const float *g = proj + (size_t)row * ldp + d.g_at() + h * d.vdim_p;
-    for (int j = lane; j < d.vdim; j += 32) store_from_float(out + (size_t)unit * d.vdim_p + j, o[j] * rn * norm[j] * silu_f(g[j]));
+#pragma unroll
+    for (int c = 0; c < 2; ++c) { // columns past vdim hold zeros
+        const int j = lane * 4 + 128 * c;
+        v[c] = j < d.vdim_p ? __ldcs(reinterpret_cast<const float4 *>(o + j)) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s += (v[c].x * v[c].x + v[c].y * v[c].y) + (v[c].z * v[c].z + v[c].w * v[c].w);
+    }
+    for (int j = 256 + lane; j < d.vdim_p; j += 32) s = fmaf(o[j], o[j], s);
+    const float rn = 1.0f / sqrtf(warp_sum(s) / (float)d.vdim + d.eps);
+    T *y = out + (size_t)unit * d.vdim_p;
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+        const int j = lane * 4 + 128 * c;
+        if (j >= d.vdim_p) continue;
+        const float4 gg = __ldcs(reinterpret_cast<const float4 *>(g + j));
+        const float e[4] = {v[c].x * silu_f(gg.x), v[c].y * silu_f(gg.y), v[c].z * silu_f(gg.z), v[c].w * silu_f(gg.w)};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) store_from_float(y + j + i, j + i < d.vdim ? e[i] * rn * norm[j + i] : 0.0f);
+    }
+    for (int j = 256 + lane; j < d.vdim; j += 32) store_from_float(y + j, o[j] * rn * norm[j] * silu_f(g[j]));
 }
 
 }  // namespace
@@ -320,23 +480,42 @@ int launch_delta_step(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float
 int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const DeltaWeights &w,
                         float *conv_state, float *state, const RowMap &rows, const SeqMap &sm, int n_rows, const int *row_seq, float *conv,
                         float *heads_out, void *out) {
+    if (d.dim_p > 256) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
+    if (n_rows > 8 * 65535 || sm.n_seq > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: too many rows or sequences in a pass");
+    if (ldp & 3) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: projection rows must keep 16-byte alignment");
     PREFER_SMEM_ONCE(delta_conv_kernel);
-    launch_pdl(ctx, delta_conv_kernel, dim3(n_rows), dim3(256), 0, d, proj, ldp, w, conv_state, rows, sm, row_seq, conv);
+    launch_pdl(ctx, delta_conv_kernel, dim3(d.kv_heads + d.heads, (n_rows + 8 * CONV_ROWS - 1) / (8 * CONV_ROWS)), dim3(256), 0, d, proj, ldp, w,
+               conv_state, rows, sm, row_seq, n_rows, conv);
     CK_LAUNCH(ctx, "delta_conv_kernel");
-    const dim3 grid(d.vdim_p / 16, d.heads, sm.n_seq);
-#define DSCAN(M)                                                                                                              \
-    do {                                                                                                                      \
-        PREFER_SMEM_ONCE(delta_scan_kernel<M>);                                                                               \
-        launch_pdl(ctx, delta_scan_kernel<M>, grid, dim3(128), 0, d, proj, ldp, conv, conv_state, state, sm, heads_out);      \
-    } while (0)
+    // columns per lane: two when that leaves every SM a dozen warps, else one (more parallel, more instructions)
+    const long long columns = (long long)d.vdim_p * d.heads * sm.n_seq;
     const int dm = (d.dim_p + 31) / 32;
-    if (dm <= 1) DSCAN(1);
-    else if (dm <= 2) DSCAN(2);
-    else if (dm <= 3) DSCAN(3);
-    else if (dm <= 4) DSCAN(4);
-    else if (dm <= 6) DSCAN(6);
-    else if (dm <= 8) DSCAN(8);
-    else return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
+    const int nc = dm > 4 ? 1 : ctx->delta_cols ? ctx->delta_cols : columns >= 4LL * 2 * 10 * ctx->sm_count ? 2 : 1;
+#define DSCAN(M, C)                                                                                                           \
+    do {                                                                                                                      \
+        constexpr int ch = M <= 4 ? 16 : 8;                                                                                   \
+        constexpr size_t smem = 2 * sizeof(float) * ch * (2 * M * 32 + 16 * C + 4);                                           \
+        static bool done[16] = {};                                                                                            \
+        if (!done[ctx->device & 15]) {                                                                                        \
+            CK(ctx, cudaFuncSetAttribute(delta_scan_kernel<M, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));   \
+            prefer_max_smem(delta_scan_kernel<M, C>);                                                                         \
+            done[ctx->device & 15] = true;                                                                                    \
+        }                                                                                                                     \
+        CK(ctx, launch_pdl(ctx, delta_scan_kernel<M, C>, dim3((d.vdim_p + 16 * C - 1) / (16 * C), d.heads, sm.n_seq),         \
+                           dim3(128), smem, d, proj, ldp, conv, conv_state, state, sm, heads_out));                           \
+    } while (0)
+#define DSCAN_C(M)                                                                                                            \
+    do {                                                                                                                      \
+        if (nc == 2) DSCAN(M, 2);                                                                                             \
+        else DSCAN(M, 1);                                                                                                     \
+    } while (0)
+    if (dm <= 1) DSCAN_C(1);
+    else if (dm <= 2) DSCAN_C(2);
+    else if (dm <= 3) DSCAN_C(3);
+    else if (dm <= 4) DSCAN_C(4);
+    else if (dm <= 6) DSCAN(6, 1);
+    else DSCAN(8, 1);
+#undef DSCAN_C
 #undef DSCAN
     CK_LAUNCH(ctx, "delta_scan_kernel");
     const int units = n_rows * d.heads;

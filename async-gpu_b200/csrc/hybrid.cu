@@ -302,7 +302,7 @@ struct b200nn_hybrid : b200nn_lm {
 int b200nn_hybrid::build_delta(const std::string &p, const LayerSpec &l, const TensorMap &t, LayerWeights *lw) {
     const DeltaDims &D = l.delta;
     const size_t KH = D.kv_heads, H = D.heads;
-    HostMat in(D.proj_w(), dp), conv(D.conv_w(), D.taps);
+    HostMat in(D.proj_w(), dp), conv(D.taps, D.conv_w());
     struct Part { const char *name; size_t heads, dim, dim_p, at; bool conv; };
     const Part parts[] = {{"q", KH, (size_t)D.dim, (size_t)D.dim_p, (size_t)D.q_at(), true},
                           {"k", KH, (size_t)D.dim, (size_t)D.dim_p, (size_t)D.k_at(), true},
@@ -317,7 +317,7 @@ int b200nn_hybrid::build_delta(const std::string &p, const LayerSpec &l, const T
         for (size_t h = 0; h < q.heads; ++h)
             for (size_t j = 0; j < q.dim; ++j) {
                 in.put(q.at + h * q.dim_p + j, m + (h * q.dim + j) * d, d);
-                if (c) conv.put(q.at + h * q.dim_p + j, c + (h * q.dim + j) * D.taps, D.taps);
+                for (int t = 0; c && t < D.taps; ++t) conv.row(t)[q.at + h * q.dim_p + j] = c[(h * q.dim + j) * D.taps + t];
             }
     }
     TRY(linear(in, &lw->in));
@@ -415,7 +415,7 @@ int b200nn_hybrid::build(const TensorMap &t) {
         if (l.type == MIX_DELTA) {
             max_proj = std::max(max_proj, (size_t)l.delta.proj_w());
             max_att = std::max(max_att, (size_t)l.delta.heads * l.delta.vdim_p);
-            max_conv = std::max(max_conv, (size_t)l.delta.conv_w() + 2 * l.delta.heads);
+            max_conv = std::max(max_conv, (size_t)l.delta.conv_ld());
             max_heads = std::max(max_heads, (size_t)l.delta.heads * l.delta.vdim_p);
         } else {
             max_proj = std::max(max_proj, up((size_t)l.lat.q_rank + l.lat.rank + l.lat.rot + l.lat.heads, 4));

@@ -66,10 +66,15 @@ struct DeltaDims {
     HD int g_at() const { return conv_w(); }
     HD int b_at() const { return g_at() + heads * vdim_p; }
     HD int a_at() const { return b_at() + heads; }
-    HD int proj_w() const { return b_at() + 2 * heads; }
+    HD int proj_w() const { return (b_at() + 2 * heads + 3) & ~3; } // rows keep 16-byte alignment
+    // convolved rows of a prompt pass (delta_rule.cu)
+    HD int decay_at() const { return conv_w(); }
+    HD int beta_at() const { return conv_w() + heads; }
+    HD int kq_at() const { return conv_w() + 2 * heads; }
+    HD int conv_ld() const { return (conv_w() + 2 * heads + kv_heads + 3) & ~3; }
 };
 struct DeltaWeights {
-    const float *conv;    // [conv_w][taps]
+    const float *conv;    // [taps][conv_w]
     const float *a_exp;   // exp(A_log) [heads]
     const float *dt_bias; // [heads]
     const float *norm;    // [vdim]
@@ -77,7 +82,7 @@ struct DeltaWeights {
 // One token of every row: convolution, unit norms, decay, state update, read-out, output norm and gate.
 int launch_delta_step(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const DeltaWeights &w, float *conv_state,
                       float *state, const RowMap &rows, int n_rows, void *out);
-// Prompt rows.  conv: [n_rows][conv_w + 2 heads] f32 (q scaled, k, v, then decay and step size), heads_out:
+// Prompt rows.  conv: [n_rows][conv_ld] f32 scratch, heads_out:
 // [n_rows][heads*vdim_p] f32 read-outs before their norm.
 int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const DeltaWeights &w,
                         float *conv_state, float *state, const RowMap &rows, const SeqMap &sm, int n_rows, const int *row_seq, float *conv,

@@ -136,6 +136,12 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_c, const __grid_c
         }
         tc::fence_mbar_init();
     }
+    if (tid == 32) {
+        tc::prefetch_tmap(&tm_c);
+        tc::prefetch_tmap(&tm_r);
+        tc::prefetch_tmap(&tm_ql);
+        tc::prefetch_tmap(&tm_qr);
+    }
     pdl_wait();
     if (warp == 1) tc::tmem_alloc(tc::smem_u32(&tmem_slot), cols);
     tc::tc_fence_before_sync();

@@ -368,35 +368,36 @@ def hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak):
     fl = pairs * 2 * (2 * dim + rot)
     out["latent_prefill_tc_kernel"] = {"tokens": T, "us": round(us, 1), "tflops": round(fl / us / 1e6, 1), "frac_of_bf16_peak": round(fl / us / 1e6 / tf_peak, 4)}
     del q, kv, rows, o
-    # latent attention, decoding with a full window
+    # latent attention, decoding with a full window: the size's own batch, and 256 sequences
     ring = -(-(window + 128) // 128) * 128
-    nbytes = batch * window * (rank + rot) * 2 + batch * H * (2 * rank + dim + rot) * 2
-    copies = max(2, int(300e6 // (batch * ring * (rank + rot) * 2)) + 1)
-    caches = [torch.randn(batch, ring, rank + rot, device=dev).to(torch.bfloat16) for _ in range(copies)]
-    q = torch.randn(batch, H * (dim + rot), device=dev).to(torch.bfloat16)
-    ql = torch.randn(batch, H * rank, device=dev).to(torch.bfloat16)
-    o = torch.empty_like(ql)
-    pos = ints([window + 5 + b % 100 for b in range(batch)])
-    call = lambda i: ops.latent_decode_attention(lat, q.data_ptr(), ql.data_ptr(), caches[i % copies].data_ptr(), ring, pos.data_ptr(), None, batch, batch,
-                                                 window + 128, o.data_ptr(), reg)
-    torch.cuda.synchronize()
-    call(0)
-    reg.synchronize()
-    us = _graph_time(reg, stream, call, 6 * copies)
-    out["latent_decode"] = {"rows": batch, "window": window, "us": round(us, 1), "GBps": round(nbytes / us / 1e3, 1),
-                            "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
-    del caches
+    for nb in (batch, 256):
+        nbytes = nb * window * (rank + rot) * 2 + nb * H * (2 * rank + dim + rot) * 2
+        copies = max(2, int(300e6 // (nb * ring * (rank + rot) * 2)) + 1)
+        caches = [torch.randn(nb, ring, rank + rot, device=dev).to(torch.bfloat16) for _ in range(copies)]
+        q = torch.randn(nb, H * (dim + rot), device=dev).to(torch.bfloat16)
+        ql = torch.randn(nb, H * rank, device=dev).to(torch.bfloat16)
+        o = torch.empty_like(ql)
+        pos = ints([window + 5 + b % 100 for b in range(nb)])
+        call = lambda i: ops.latent_decode_attention(lat, q.data_ptr(), ql.data_ptr(), caches[i % copies].data_ptr(), ring, pos.data_ptr(), None,
+                                                     nb, nb, window + 128, o.data_ptr(), reg)
+        torch.cuda.synchronize()
+        call(0)
+        reg.synchronize()
+        us = _graph_time(reg, stream, call, 6 * copies)
+        out[f"latent_decode_tc_kernel_rows{nb}"] = {"us": round(us, 1), "MB": round(nbytes / 1e6, 1), "GBps": round(nbytes / us / 1e3, 1),
+                                                    "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
+        del caches
     # delta rule
     sh = (H, KH, dim, dim, 4, 1e-5)
     cw = 2 * KH * dim + H * dim
-    pw = cw + H * dim + 2 * H
-    wts = [torch.randn(cw, 4, device=dev), torch.full((H,), 0.1, device=dev), torch.zeros(H, device=dev), torch.ones(dim, device=dev)]
+    pw = -(-(cw + H * dim + 2 * H) // 4) * 4
+    wts = [torch.randn(4, cw, device=dev), torch.full((H,), 0.1, device=dev), torch.zeros(H, device=dev), torch.ones(dim, device=dev)]
     ptrs = tuple(t.data_ptr() for t in wts)
     proj = torch.randn(max(T, batch), pw, device=dev)
     conv = torch.zeros(batch, 4, cw, device=dev)
     state = torch.zeros(batch, H, dim, dim, device=dev)
     o = torch.empty(max(T, batch), H * dim, device=dev, dtype=torch.bfloat16)
-    scratch = torch.empty(T * (cw + 2 * H + H * dim), device=dev)
+    scratch = torch.empty(T * (cw + 2 * H + KH + 4 + H * dim), device=dev)
     rpos, rslot = ints([i % prompt for i in range(T)]), ints([i // prompt for i in range(T)])
     seq = ints(range(B), r0, [prompt] * B, [0] * B, [i // prompt for i in range(T)])
     call = lambda i: ops.delta_rule(sh, ptrs, proj.data_ptr(), conv.data_ptr(), state.data_ptr(), rpos.data_ptr(), rslot.data_ptr(), T, o.data_ptr(),
@@ -408,16 +409,21 @@ def hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak):
     fl = 6 * dim * dim * H * T
     out["delta_prompt"] = {"tokens": T, "sequences": B, "us": round(us, 1), "tflops_f32": round(fl / us / 1e6, 2),
                            "frac_of_f32_peak": round(fl / us / 1e6 / f32_peak, 4)}
-    copies = max(2, int(300e6 // (state.numel() * 4)) + 1)
-    states = [torch.randn_like(state) * 0.01 for _ in range(copies)]
-    pos = ints([100] * batch)
-    call = lambda i: ops.delta_rule(sh, ptrs, proj.data_ptr(), conv.data_ptr(), states[i % copies].data_ptr(), pos.data_ptr(), None, batch, o.data_ptr(), reg)
-    torch.cuda.synchronize()
-    call(0)
-    reg.synchronize()
-    us = _graph_time(reg, stream, call, 6 * copies)
-    nbytes = 2 * state.numel() * 4 + batch * pw * 4 + batch * 4 * cw * 4 + batch * H * dim * 2
-    out["delta_step_kernel"] = {"rows": batch, "us": round(us, 1), "GBps": round(nbytes / us / 1e3, 1), "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
+    for nb in (batch, 256):
+        state = torch.zeros(nb, H, dim, dim, device=dev)
+        conv = torch.zeros(nb, 4, cw, device=dev)
+        copies = max(2, int(300e6 // (state.numel() * 4)) + 1)
+        states = [torch.randn_like(state) * 0.01 for _ in range(copies)]
+        pos = ints([100] * nb)
+        call = lambda i: ops.delta_rule(sh, ptrs, proj.data_ptr(), conv.data_ptr(), states[i % copies].data_ptr(), pos.data_ptr(), None, nb, o.data_ptr(), reg)
+        torch.cuda.synchronize()
+        call(0)
+        reg.synchronize()
+        us = _graph_time(reg, stream, call, 6 * copies)
+        nbytes = 2 * state.numel() * 4 + nb * pw * 4 + nb * 4 * cw * 4 + nb * H * dim * 2
+        out[f"delta_step_kernel_rows{nb}"] = {"us": round(us, 1), "MB": round(nbytes / 1e6, 1), "GBps": round(nbytes / us / 1e3, 1),
+                                              "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
+        del states
     return out
 
 

@@ -135,6 +135,7 @@ B200NN_API int32_t b200nn_ctx_set_gemv_max_rows(b200nn_ctx *ctx, int32_t rows);
  * (the residual GEMMs then need complete sums, i.e. cluster splits); sessions read it when created.
  * "lm_portion" (default 0 = 2048): most new tokens of one sequence a hybrid model's cache takes in a pass; a
  * windowed layer's ring holds the window plus this many rows.  Read when a cache or session is created.
+ * "delta_cols" (default 0 = by the amount of work): state columns per lane of the delta rule's prompt kernel (1 or 2).
  * "persist" (default 0): decode steps of an int4 model run all transformer blocks as one cooperative
  * kernel (decode sessions whose shape it supports).  Measured slower than the per-op CUDA graph.
  * Its aids: "persist_min_rows" / "persist_max_rows" (batch range it is used for), "persist_prefetch_mb",
@@ -576,12 +577,12 @@ B200NN_API int32_t b200nn_latent_decode_attention(b200nn_ctx *ctx, const b200nn_
                                                   const int32_t *slot_dev, int32_t n_slots, int32_t n_rows, int32_t capacity,
                                                   void *out_dev);
 /* Gated delta rule with its short convolution, norms and output gate.  proj f32 [n_rows] x ([kv_heads][dim] q,
- * [kv_heads][dim] k, [heads][vdim] v, [heads][vdim] gate, [heads] step-size and [heads] decay inputs); weights
- * f32 on the device: conv [2 kv_heads dim + heads vdim][conv taps], a_exp [heads] = exp(A_log), dt_bias [heads],
+ * [kv_heads][dim] k, [heads][vdim] v, [heads][vdim] gate, [heads] step-size and [heads] decay inputs, then padding to a multiple of 4); weights
+ * f32 on the device: conv [taps][2 kv_heads dim + heads vdim], a_exp [heads] = exp(A_log), dt_bias [heads],
  * norm [vdim]; conv_state f32 [slots][taps][2 kv_heads dim + heads vdim], state f32 [slots][heads][dim][vdim];
  * out [n_rows][heads][vdim].  n_seq 0: one token per row.  Else prompt portions: seq [4][n_seq] (slot, first row,
  * rows, past) followed by the sequence index of every row, slot per row given, and scratch f32 of
- * n_rows * (2 kv_heads dim + 2 heads vdim + 2 heads). */
+ * n_rows * (2 kv_heads dim + 2 heads vdim + 2 heads + kv_heads + 4). */
 typedef struct {
     int32_t heads, kv_heads, dim, vdim, conv;
     float eps;

@@ -395,8 +395,18 @@ def test_latent_decode_attention(reg, shape, spike, dtype):
     assert reg.device_error() == 0
 
 
-@pytest.mark.parametrize("shape", [(4, 2, 32, 48, 4), (2, 2, 128, 128, 3), (3, 1, 64, 16, 1), (1, 1, 96, 208, 2), (2, 1, 176, 32, 6)])
-def test_delta_rule(reg, shape):
+@pytest.mark.parametrize("shape", [(4, 2, 32, 48, 4), (2, 2, 128, 128, 3), (3, 1, 64, 16, 1), (1, 1, 96, 208, 2), (2, 1, 176, 32, 6),
+                                   (64, 16, 64, 128, 2)])
+@pytest.mark.parametrize("cols", [0, 1, 2])
+def test_delta_rule(reg, shape, cols):
+    reg.set_tuning("delta_cols", cols)
+    try:
+        delta_rule_case(reg, shape)
+    finally:
+        reg.set_tuning("delta_cols", 0)
+
+
+def delta_rule_case(reg, shape):
     """Prompt portions, then single tokens, on ragged sequences; outputs and the states they leave.  Decays from
     instant forgetting to none, so that a state that is lost, doubled or shifted shows."""
     import torch
@@ -404,12 +414,13 @@ def test_delta_rule(reg, shape):
     rng = np.random.default_rng(sum(shape))
     eps = 1e-5
     pw = 2 * KH * dim + 2 * H * vdim + 2 * H
+    pad = -pw % 4
     cw = 2 * KH * dim + H * vdim
     lens = [1, 2, 5, 33, 100, 257]
     E = len(lens)
     proj = [rng.standard_normal((n + 3, pw)).astype(np.float32) for n in lens]
     conv = rng.standard_normal((cw, taps)).astype(np.float32)
-    a_log = np.linspace(-6.0, 2.0, H)
+    a_log = np.linspace(-6.0, 3.0, H)
     dt = rng.uniform(-3, 1, H).astype(np.float32)
     norm = rng.uniform(0.5, 1.5, vdim).astype(np.float32)
 
@@ -432,14 +443,14 @@ def test_delta_rule(reg, shape):
     slots = rng.permutation(E + 1)[:E]
     cs = torch.full((E + 1, taps, cw), float("nan"), device="cuda")
     st = torch.full((E + 1, H, dim, vdim), float("nan"), device="cuda")
-    wt = [_dev(conv), _dev(np.exp(a_log)), _dev(dt), _dev(norm)]
+    wt = [_dev(conv.T), _dev(np.exp(a_log)), _dev(dt), _dev(norm)]
     ptrs = tuple(t.data_ptr() for t in wt)
     got = [[] for _ in lens]
     at = [0] * E
     for cut in (0.4, 1.0):  # two portions
         part = [(i, at[i], max(at[i], int(np.ceil(n * cut)))) for i, n in enumerate(lens)]
         part = [(i, a, b) for i, a, b in part if b > a]
-        rows = np.concatenate([proj[i][a:b] for i, a, b in part])
+        rows = np.pad(np.concatenate([proj[i][a:b] for i, a, b in part]), ((0, 0), (0, pad)))
         pos = np.concatenate([np.arange(a, b) for _, a, b in part])
         sl = np.concatenate([np.full(b - a, slots[i]) for i, a, b in part])
         n = [b - a for _, a, b in part]
@@ -447,7 +458,7 @@ def test_delta_rule(reg, shape):
         meta = _ints([slots[i] for i, _, _ in part], row0, n, [a for _, a, _ in part], np.repeat(np.arange(len(part)), n))
         tp, tpos, tsl = _dev(rows), _ints(pos), _ints(sl)
         out = torch.zeros((len(rows), H, vdim), device="cuda")
-        scratch = torch.empty(len(rows) * (cw + 2 * H + H * vdim), device="cuda")
+        scratch = torch.empty(len(rows) * (cw + 2 * H + KH + 4 + H * vdim), device="cuda")
         torch.cuda.synchronize()
         ops.delta_rule((H, KH, dim, vdim, taps, eps), ptrs, tp.data_ptr(), cs.data_ptr(), st.data_ptr(), tpos.data_ptr(), tsl.data_ptr(), len(rows),
                        out.data_ptr(), reg, len(part), max(n), meta.data_ptr(), scratch.data_ptr(), flags=b200nn.LM_F32)
@@ -457,7 +468,7 @@ def test_delta_rule(reg, shape):
             got[i].append(o[r:r + b - a])
             at[i] = b
     for step in range(3):
-        tp, tpos, tsl = _dev(np.stack([proj[i][lens[i] + step] for i in range(E)])), _ints([n + step for n in lens]), _ints(slots)
+        tp, tpos, tsl = _dev(np.pad(np.stack([proj[i][lens[i] + step] for i in range(E)]), ((0, 0), (0, pad)))), _ints([n + step for n in lens]), _ints(slots)
         out = torch.zeros((E, H, vdim), device="cuda")
         torch.cuda.synchronize()
         ops.delta_rule((H, KH, dim, vdim, taps, eps), ptrs, tp.data_ptr(), cs.data_ptr(), st.data_ptr(), tpos.data_ptr(), tsl.data_ptr(), E,
