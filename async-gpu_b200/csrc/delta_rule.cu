@@ -24,14 +24,16 @@ __device__ __forceinline__ float decay_f(float a_exp, float a, float dt_bias) { 
 
 // ---- decoding ----------------------------------------------------------------------------------------
 // Block = (row, head), eight warps.  Warp w holds state rows w, w + 8, ...; lane l columns 4l .. 4l+3 of a
-// 128-column chunk (one chunk for vdim <= 128).
+// 128-column chunk (one chunk for vdim <= 128).  Under the state's loads warp 0 makes the query and key (a lane takes
+// four channels; their norms stay scalar factors), warp 1 the value, warp 2 gate times norm weight, warp 3 decay and
+// step size.
 template <int RPW, typename T>
 __global__ void __launch_bounds__(256)
 delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWeights w, float *__restrict__ conv_state,
                   float *__restrict__ state, RowMap rows, T *__restrict__ out) {
-    extern __shared__ float sh[]; // q [dim_p], k [dim_p], v [vdim_p], o [vdim_p], reduction [8][2][128], scalars [8]
+    extern __shared__ __align__(16) float sh[]; // q [dim_p], k [dim_p], v, gate, o [vdim_p], reduction [8][2][128], scalars [8]
     const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    float *sq = sh, *sk = sq + d.dim_p, *sv = sk + d.dim_p, *so = sv + d.vdim_p, *red = so + d.vdim_p, *sc = red + 2048;
+    float *sq = sh, *sk = sq + d.dim_p, *sv = sk + d.dim_p, *sgn = sv + d.vdim_p, *so = sgn + d.vdim_p, *red = so + d.vdim_p, *sc = red + 2048;
     pdl_trigger();
     pdl_wait();
     const int pos = row_pos(rows, row), slot = row_slot(rows, row);
@@ -42,7 +44,7 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
 #pragma unroll
         for (int r = 0; r < RPW; ++r) {
             const int i = warp + 8 * r;
-            st[r] = col && i < d.dim_p && pos > 0 ? *reinterpret_cast<const float4 *>(S + (size_t)i * d.vdim_p + c0 + lane * 4)
+            st[r] = col && i < d.dim_p && pos > 0 ? __ldcs(reinterpret_cast<const float4 *>(S + (size_t)i * d.vdim_p + c0 + lane * 4))
                                                   : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     };
@@ -50,38 +52,51 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
 
     const float *p = proj + (size_t)row * ldp;
     const int group = d.heads / d.kv_heads, kh = h / group;
-    const int cw = d.conv_w();
+    const int cw = d.conv_w(), here = pos % d.taps;
     float *cring = conv_state + (size_t)slot * d.taps * cw;
-    for (int t = tid; t < 2 * d.dim_p + d.vdim_p; t += 256) {
-        const int which = t < d.dim_p ? 0 : t < 2 * d.dim_p ? 1 : 2;
-        const int ch = which == 0 ? d.q_at() + kh * d.dim_p + t
-                                  : which == 1 ? d.k_at() + kh * d.dim_p + (t - d.dim_p) : d.v_at() + h * d.vdim_p + (t - 2 * d.dim_p);
-        const float x = p[ch];
-        const float *cwt = w.conv + ch;
-        float a = x * cwt[(size_t)(d.taps - 1) * cw];
-        for (int j = 1; j < d.taps; ++j)
-            if (pos - j >= 0) a = fmaf(cring[(size_t)((pos - j) % d.taps) * cw + ch], cwt[(size_t)(d.taps - 1 - j) * cw], a);
-        if (which == 2 || h % group == 0) cring[(size_t)(pos % d.taps) * cw + ch] = x;
-        sh[t] = silu_f(a); // q, k and v lie behind one another
-    }
-    __syncthreads();
-    if (warp < 2) { // unit norms; q also times dim^(-1/2)
-        float *x = warp ? sk : sq;
-        float s = 0.0f;
-        for (int j = lane; j < d.dim_p; j += 32) s = fmaf(x[j], x[j], s);
-        s = warp_sum(s);
-        float f = 1.0f / sqrtf(s + 1e-6f);
-        if (warp == 0) f *= 1.0f / sqrtf((float)d.dim);
-        for (int j = lane; j < d.dim_p; j += 32) x[j] *= f;
-    } else if (tid == 64) {
+    auto channels = [&](int ch, bool keep) { // four channels after convolution and silu; keep: put the input into the ring
+        const float4 x = *reinterpret_cast<const float4 *>(p + ch), w0 = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1) * cw + ch));
+        float4 a = make_float4(x.x * w0.x, x.y * w0.y, x.z * w0.z, x.w * w0.w);
+#pragma unroll 4
+        for (int t = 1; t < d.taps; ++t)
+            if (pos - t >= 0) {
+                const int at = here - t < 0 ? here - t + d.taps : here - t;
+                const float4 y = *reinterpret_cast<const float4 *>(cring + (size_t)at * cw + ch);
+                const float4 wt = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1 - t) * cw + ch));
+                a.x = fmaf(y.x, wt.x, a.x); a.y = fmaf(y.y, wt.y, a.y); a.z = fmaf(y.z, wt.z, a.z); a.w = fmaf(y.w, wt.w, a.w);
+            }
+        if (keep) *reinterpret_cast<float4 *>(cring + (size_t)here * cw + ch) = x;
+        return make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
+    };
+    if (warp == 0) {
+        float qq = 0.0f, kk = 0.0f, kq = 0.0f;
+        for (int j = lane * 4; j < d.dim_p; j += 128) {
+            const float4 a = channels(d.q_at() + kh * d.dim_p + j, h % group == 0), b = channels(d.k_at() + kh * d.dim_p + j, h % group == 0);
+            *reinterpret_cast<float4 *>(sq + j) = a;
+            *reinterpret_cast<float4 *>(sk + j) = b;
+            qq += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
+            kk += (b.x * b.x + b.y * b.y) + (b.z * b.z + b.w * b.w);
+            kq += (a.x * b.x + a.y * b.y) + (a.z * b.z + a.w * b.w);
+        }
+        qq = warp_sum(qq);
+        kk = warp_sum(kk);
+        kq = warp_sum(kq);
+        if (lane == 0) { // unit norms; q also times dim^(-1/2)
+            const float fq = 1.0f / sqrtf(qq + 1e-6f) / sqrtf((float)d.dim), fk = 1.0f / sqrtf(kk + 1e-6f);
+            sc[2] = fq;
+            sc[3] = fk;
+            sc[4] = kq * fq * fk;
+        }
+    } else if (warp == 1) {
+        for (int j = lane * 4; j < d.vdim_p; j += 128) *reinterpret_cast<float4 *>(sv + j) = channels(d.v_at() + h * d.vdim_p + j, true);
+    } else if (warp == 2) {
+        for (int j = lane; j < d.vdim; j += 32) sgn[j] = w.norm[j] * silu_f(p[d.g_at() + h * d.vdim_p + j]);
+    } else if (tid == 96) {
         sc[0] = sigmoid_f(p[d.b_at() + h]);
         sc[1] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
     }
     __syncthreads();
-    float kq = 0.0f;
-    for (int j = lane; j < d.dim_p; j += 32) kq = fmaf(sk[j], sq[j], kq);
-    kq = warp_sum(kq);
-    const float beta = sc[0], g = sc[1];
+    const float beta = sc[0], g = sc[1], fq = sc[2], fk = sc[3], kq = sc[4];
     for (int c0 = 0; c0 < d.vdim_p; c0 += 128) {
         if (c0) load_chunk(c0);
         float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
@@ -99,35 +114,36 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         __syncthreads();
         float4 tk = make_float4(0.f, 0.f, 0.f, 0.f), tq = tk;
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            tk = f4_add(tk, *reinterpret_cast<const float4 *>(red + (i * 2) * 128 + lane * 4));
-            tq = f4_add(tq, *reinterpret_cast<const float4 *>(red + (i * 2 + 1) * 128 + lane * 4));
-        }
+        for (int i = 0; i < 8; ++i) tk = f4_add(tk, *reinterpret_cast<const float4 *>(red + (i * 2) * 128 + lane * 4));
+        if (warp == 0)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) tq = f4_add(tq, *reinterpret_cast<const float4 *>(red + (i * 2 + 1) * 128 + lane * 4));
         const int c = c0 + lane * 4;
         if (c < d.vdim_p) {
             const float4 v = *reinterpret_cast<const float4 *>(sv + c);
-            const float4 u = make_float4(beta * (v.x - g * tk.x), beta * (v.y - g * tk.y), beta * (v.z - g * tk.z), beta * (v.w - g * tk.w));
-            if (warp == 0)
-                *reinterpret_cast<float4 *>(so + c) =
-                    make_float4(fmaf(kq, u.x, g * tq.x), fmaf(kq, u.y, g * tq.y), fmaf(kq, u.z, g * tq.z), fmaf(kq, u.w, g * tq.w));
+            const float gk = g * fk, gq = g * fq;
+            const float4 u = make_float4(beta * (v.x - gk * tk.x), beta * (v.y - gk * tk.y), beta * (v.z - gk * tk.z), beta * (v.w - gk * tk.w));
 #pragma unroll
             for (int r = 0; r < RPW; ++r) {
                 const int i = warp + 8 * r;
                 if (i < d.dim_p) {
-                    const float k = sk[i];
-                    *reinterpret_cast<float4 *>(S + (size_t)i * d.vdim_p + c) =
-                        make_float4(fmaf(k, u.x, g * st[r].x), fmaf(k, u.y, g * st[r].y), fmaf(k, u.z, g * st[r].z), fmaf(k, u.w, g * st[r].w));
+                    const float k = sk[i] * fk;
+                    __stcs(reinterpret_cast<float4 *>(S + (size_t)i * d.vdim_p + c),
+                           make_float4(fmaf(k, u.x, g * st[r].x), fmaf(k, u.y, g * st[r].y), fmaf(k, u.z, g * st[r].z), fmaf(k, u.w, g * st[r].w)));
                 }
             }
+            if (warp == 0)
+                *reinterpret_cast<float4 *>(so + c) =
+                    make_float4(fmaf(kq, u.x, gq * tq.x), fmaf(kq, u.y, gq * tq.y), fmaf(kq, u.z, gq * tq.z), fmaf(kq, u.w, gq * tq.w));
         }
-        __syncthreads();
+        if (c0 + 128 < d.vdim_p) __syncthreads(); // red is used again
     }
-    float s = 0.0f; // every warp takes the sum for itself
+    if (warp) return; // the read-out is warp 0's own
+    __syncwarp();
+    float s = 0.0f;
     for (int j = lane; j < d.vdim; j += 32) s = fmaf(so[j], so[j], s);
-    s = warp_sum(s);
-    const float rn = 1.0f / sqrtf(s / (float)d.vdim + d.eps);
-    for (int j = tid; j < d.vdim; j += 256)
-        store_from_float(out + ((size_t)row * d.heads + h) * d.vdim_p + j, so[j] * rn * w.norm[j] * silu_f(p[d.g_at() + h * d.vdim_p + j]));
+    const float rn = 1.0f / sqrtf(warp_sum(s) / (float)d.vdim + d.eps);
+    for (int j = lane; j < d.vdim; j += 32) store_from_float(out + ((size_t)row * d.heads + h) * d.vdim_p + j, so[j] * rn * sgn[j]);
 }
 
 // ---- prompts -----------------------------------------------------------------------------------------
@@ -456,7 +472,7 @@ int launch_delta_step(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float
                       float *state, const RowMap &rows, int n_rows, void *out) {
     if (n_rows > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: more than 65535 rows");
     const dim3 grid(d.heads, n_rows);
-    const size_t smem = (2 * d.dim_p + 2 * d.vdim_p + 2048 + 8) * sizeof(float);
+    const size_t smem = (2 * d.dim_p + 3 * d.vdim_p + 2048 + 8) * sizeof(float);
 #define DSTEP(R)                                                                                                             \
     do {                                                                                                                     \
         PREFER_SMEM_ONCE((delta_step_kernel<R, __nv_bfloat16>));                                                             \
