@@ -24,11 +24,11 @@ __device__ __forceinline__ float decay_f(float a_exp, float a, float dt_bias) { 
 
 // ---- decoding ----------------------------------------------------------------------------------------
 // Block = (row, head), eight warps.  Warp w holds state rows w, w + 8, ...; lane l columns 4l .. 4l+3 of a
-// 128-column chunk (one chunk for vdim <= 128).  Under the state's loads warp 0 makes the query and key (a lane takes
-// four channels; their norms stay scalar factors), warp 1 the value, warp 2 gate times norm weight, warp 3 decay and
+// 128-column chunk (one chunk for vdim <= 128).  Under the state's loads warps 0, 1 and 2 make the query, key and value
+// (a lane takes four channels; the unit norms stay scalar factors), warp 3 gate times norm weight, warp 4 decay and
 // step size.
 template <int RPW, typename T>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, RPW <= 16 ? 2 : 1)
 delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWeights w, float *__restrict__ conv_state,
                   float *__restrict__ state, RowMap rows, T *__restrict__ out) {
     extern __shared__ __align__(16) float sh[]; // q [dim_p], k [dim_p], v, gate, o [vdim_p], reduction [8][2][128], scalars [8]
@@ -44,7 +44,7 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
 #pragma unroll
         for (int r = 0; r < RPW; ++r) {
             const int i = warp + 8 * r;
-            st[r] = col && i < d.dim_p && pos > 0 ? __ldcs(reinterpret_cast<const float4 *>(S + (size_t)i * d.vdim_p + c0 + lane * 4))
+            st[r] = col && i < d.dim_p && pos > 0 ? *reinterpret_cast<const float4 *>(S + (size_t)i * d.vdim_p + c0 + lane * 4)
                                                   : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     };
@@ -54,49 +54,68 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
     const int group = d.heads / d.kv_heads, kh = h / group;
     const int cw = d.conv_w(), here = pos % d.taps;
     float *cring = conv_state + (size_t)slot * d.taps * cw;
-    auto channels = [&](int ch, bool keep) { // four channels after convolution and silu; keep: put the input into the ring
-        const float4 x = *reinterpret_cast<const float4 *>(p + ch), w0 = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1) * cw + ch));
-        float4 a = make_float4(x.x * w0.x, x.y * w0.y, x.z * w0.z, x.w * w0.w);
-#pragma unroll 4
-        for (int t = 1; t < d.taps; ++t)
-            if (pos - t >= 0) {
-                const int at = here - t < 0 ? here - t + d.taps : here - t;
-                const float4 y = *reinterpret_cast<const float4 *>(cring + (size_t)at * cw + ch);
-                const float4 wt = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1 - t) * cw + ch));
-                a.x = fmaf(y.x, wt.x, a.x); a.y = fmaf(y.y, wt.y, a.y); a.z = fmaf(y.z, wt.z, a.z); a.w = fmaf(y.w, wt.w, a.w);
-            }
-        if (keep) *reinterpret_cast<float4 *>(cring + (size_t)here * cw + ch) = x;
+    // four channels: the inputs of up to four taps are requested together, then summed; keep: put the input into the ring
+    struct Taps {
+        float4 x[4], w[4];
+    };
+    auto request = [&](int ch) {
+        Taps t;
+        t.x[0] = *reinterpret_cast<const float4 *>(p + ch);
+        t.w[0] = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1) * cw + ch));
+#pragma unroll
+        for (int i = 1; i < 4; ++i) {
+            const bool use = i < d.taps && pos >= i;
+            const int at = use ? (here - i < 0 ? here - i + d.taps : here - i) : here, tap = use ? d.taps - 1 - i : d.taps - 1;
+            const float4 y = *reinterpret_cast<const float4 *>(cring + (size_t)at * cw + ch);
+            t.x[i] = use ? y : make_float4(0.f, 0.f, 0.f, 0.f);
+            t.w[i] = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)tap * cw + ch));
+        }
+        return t;
+    };
+    auto channels = [&](const Taps &t, int ch, bool keep) {
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            a.x = fmaf(t.x[i].x, t.w[i].x, a.x); a.y = fmaf(t.x[i].y, t.w[i].y, a.y);
+            a.z = fmaf(t.x[i].z, t.w[i].z, a.z); a.w = fmaf(t.x[i].w, t.w[i].w, a.w);
+        }
+        for (int i = 4; i < d.taps && pos >= i; ++i) {
+            const float4 y = *reinterpret_cast<const float4 *>(cring + (size_t)(here - i < 0 ? here - i + d.taps : here - i) * cw + ch);
+            const float4 wt = __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1 - i) * cw + ch));
+            a.x = fmaf(y.x, wt.x, a.x); a.y = fmaf(y.y, wt.y, a.y); a.z = fmaf(y.z, wt.z, a.z); a.w = fmaf(y.w, wt.w, a.w);
+        }
+        if (keep) *reinterpret_cast<float4 *>(cring + (size_t)here * cw + ch) = t.x[0];
         return make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
     };
-    if (warp == 0) {
-        float qq = 0.0f, kk = 0.0f, kq = 0.0f;
-        for (int j = lane * 4; j < d.dim_p; j += 128) {
-            const float4 a = channels(d.q_at() + kh * d.dim_p + j, h % group == 0), b = channels(d.k_at() + kh * d.dim_p + j, h % group == 0);
-            *reinterpret_cast<float4 *>(sq + j) = a;
-            *reinterpret_cast<float4 *>(sk + j) = b;
-            qq += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
-            kk += (b.x * b.x + b.y * b.y) + (b.z * b.z + b.w * b.w);
-            kq += (a.x * b.x + a.y * b.y) + (a.z * b.z + a.w * b.w);
+    if (warp < 3) { // query, key, value
+        const int n = warp < 2 ? d.dim_p : d.vdim_p, at = warp == 0 ? d.q_at() + kh * d.dim_p : warp == 1 ? d.k_at() + kh * d.dim_p : d.v_at() + h * d.vdim_p;
+        float *dst = warp == 0 ? sq : warp == 1 ? sk : sv;
+        float s = 0.0f;
+        for (int j = lane * 4; j < n; j += 128) {
+            const float4 a = channels(request(at + j), at + j, warp == 2 || h % group == 0);
+            *reinterpret_cast<float4 *>(dst + j) = a;
+            s += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
         }
-        qq = warp_sum(qq);
-        kk = warp_sum(kk);
-        kq = warp_sum(kq);
-        if (lane == 0) { // unit norms; q also times dim^(-1/2)
-            const float fq = 1.0f / sqrtf(qq + 1e-6f) / sqrtf((float)d.dim), fk = 1.0f / sqrtf(kk + 1e-6f);
-            sc[2] = fq;
-            sc[3] = fk;
-            sc[4] = kq * fq * fk;
+        s = warp_sum(s);
+        if (lane == 0) sc[2 + warp] = 1.0f / sqrtf(s + 1e-6f); // unit norms (the value's is not used)
+    } else if (warp == 3) {
+        for (int j = lane * 4; j < d.vdim_p; j += 128) { // the last columns may be padding: no norm weight there
+            const float4 gg = *reinterpret_cast<const float4 *>(p + d.g_at() + h * d.vdim_p + j);
+            const float e[4] = {gg.x, gg.y, gg.z, gg.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i) sgn[j + i] = j + i < d.vdim ? w.norm[j + i] * silu_f(e[i]) : 0.0f;
         }
-    } else if (warp == 1) {
-        for (int j = lane * 4; j < d.vdim_p; j += 128) *reinterpret_cast<float4 *>(sv + j) = channels(d.v_at() + h * d.vdim_p + j, true);
-    } else if (warp == 2) {
-        for (int j = lane; j < d.vdim; j += 32) sgn[j] = w.norm[j] * silu_f(p[d.g_at() + h * d.vdim_p + j]);
-    } else if (tid == 96) {
+    } else if (tid == 128) {
         sc[0] = sigmoid_f(p[d.b_at() + h]);
         sc[1] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
     }
     __syncthreads();
-    const float beta = sc[0], g = sc[1], fq = sc[2], fk = sc[3], kq = sc[4];
+    const float beta = sc[0], g = sc[1], fq = sc[2] / sqrtf((float)d.dim), fk = sc[3]; // q also times dim^(-1/2)
+    float kq = 0.0f; // warp 0, which makes the read-out, needs k . q
+    if (warp == 0) {
+        for (int j = lane; j < d.dim_p; j += 32) kq = fmaf(sk[j], sq[j], kq);
+        kq = warp_sum(kq) * fq * fk;
+    }
     for (int c0 = 0; c0 < d.vdim_p; c0 += 128) {
         if (c0) load_chunk(c0);
         float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
@@ -128,8 +147,8 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
                 const int i = warp + 8 * r;
                 if (i < d.dim_p) {
                     const float k = sk[i] * fk;
-                    __stcs(reinterpret_cast<float4 *>(S + (size_t)i * d.vdim_p + c),
-                           make_float4(fmaf(k, u.x, g * st[r].x), fmaf(k, u.y, g * st[r].y), fmaf(k, u.z, g * st[r].z), fmaf(k, u.w, g * st[r].w)));
+                    *reinterpret_cast<float4 *>(S + (size_t)i * d.vdim_p + c) =
+                        make_float4(fmaf(k, u.x, g * st[r].x), fmaf(k, u.y, g * st[r].y), fmaf(k, u.z, g * st[r].z), fmaf(k, u.w, g * st[r].w));
                 }
             }
             if (warp == 0)
