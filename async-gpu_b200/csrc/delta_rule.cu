@@ -17,7 +17,8 @@
 
 namespace {
 
-__device__ __forceinline__ float silu_f(float v) { return v / (1.0f + expf(-v)); }
+// activation of the convolution and of the output gate (not part of the recurrence): fast exponential and division
+__device__ __forceinline__ float silu_f(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
 __device__ __forceinline__ float decay_f(float a_exp, float a, float dt_bias) { return expf(-a_exp * softplus_f(a + dt_bias)); }
@@ -171,7 +172,9 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
 //
 // A warp takes four rows of one unit: a query/key head (both of its vectors) or a value head.  The eight warps of a
 // block take neighbouring rows, which share their convolution inputs in L1.
+// NCH: 128-channel chunks of a query/key head.
 constexpr int CONV_ROWS = 4;
+template <int NCH>
 __global__ void __launch_bounds__(256)
 delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWeights w, const float *__restrict__ conv_state, RowMap rows,
                   SeqMap sm, const int *__restrict__ row_seq, int n_rows, float *__restrict__ conv) {
@@ -200,12 +203,36 @@ delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         }
         return make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
     };
+    // the same for all four rows; four neighbours of one sequence with their inputs in the pass share seven loads
+    const bool shared = d.taps <= 4 && back[0] >= 3 && back[CONV_ROWS - 1] == back[0] + CONV_ROWS - 1 && r_first + CONV_ROWS <= n_rows;
+    auto rows4 = [&](int ch, float4 (&o)[CONV_ROWS]) {
+        if (!shared) {
+#pragma unroll
+            for (int r = 0; r < CONV_ROWS; ++r) o[r] = channels(r, ch);
+            return;
+        }
+        float4 x[CONV_ROWS + 3], wt[4];
+#pragma unroll
+        for (int i = 0; i < CONV_ROWS + 3; ++i) x[i] = *reinterpret_cast<const float4 *>(proj + (size_t)(r_first + i - 3) * ldp + ch);
+#pragma unroll
+        for (int t = 0; t < 4; ++t)
+            wt[t] = t < d.taps ? __ldg(reinterpret_cast<const float4 *>(w.conv + (size_t)(d.taps - 1 - t) * cw + ch)) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int r = 0; r < CONV_ROWS; ++r) {
+            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+                const float4 y = x[3 + r - t];
+                a.x = fmaf(y.x, wt[t].x, a.x); a.y = fmaf(y.y, wt[t].y, a.y); a.z = fmaf(y.z, wt[t].z, a.z); a.w = fmaf(y.w, wt[t].w, a.w);
+            }
+            o[r] = make_float4(silu_f(a.x), silu_f(a.y), silu_f(a.z), silu_f(a.w));
+        }
+    };
     if (u >= d.kv_heads) { // a value head
         const int h = u - d.kv_heads;
         for (int j = lane * 4; j < d.vdim_p; j += 128) {
             float4 v[CONV_ROWS];
-#pragma unroll
-            for (int r = 0; r < CONV_ROWS; ++r) v[r] = channels(r, d.v_at() + h * d.vdim_p + j);
+            rows4(d.v_at() + h * d.vdim_p + j, v);
 #pragma unroll
             for (int r = 0; r < CONV_ROWS; ++r)
                 if (r_first + r < n_rows) *reinterpret_cast<float4 *>(conv + (size_t)(r_first + r) * ld + d.v_at() + h * d.vdim_p + j) = v[r];
@@ -219,45 +246,41 @@ delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         return;
     }
     const float q_scale = 1.0f / sqrtf((float)d.dim);
+    float4 q[NCH][CONV_ROWS], k[NCH][CONV_ROWS];
 #pragma unroll
-    for (int half = 0; half < 2; ++half) { // two rows at a time
-        float4 q[2][2], k[2][2]; // [row][chunk of 128]; dim <= 256
-        float qq[2], kk[2], kq[2];
+    for (int c = 0; c < NCH; ++c) {
+        const int j = lane * 4 + 128 * c;
 #pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            qq[r] = kk[r] = kq[r] = 0.0f;
+        for (int r = 0; r < CONV_ROWS; ++r) q[c][r] = k[c][r] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < d.dim_p) {
+            rows4(d.q_at() + u * d.dim_p + j, q[c]);
+            rows4(d.k_at() + u * d.dim_p + j, k[c]);
+        }
+    }
 #pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const int j = lane * 4 + 128 * c;
-                float4 &a = q[r][c], &b = k[r][c];
-                a = b = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (j < d.dim_p) {
-                    a = channels(2 * half + r, d.q_at() + u * d.dim_p + j);
-                    b = channels(2 * half + r, d.k_at() + u * d.dim_p + j);
-                }
-                qq[r] += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
-                kk[r] += (b.x * b.x + b.y * b.y) + (b.z * b.z + b.w * b.w);
-                kq[r] += (a.x * b.x + a.y * b.y) + (a.z * b.z + a.w * b.w);
+    for (int r = 0; r < CONV_ROWS; ++r) {
+        float qq = 0.0f, kk = 0.0f, kq = 0.0f;
+#pragma unroll
+        for (int c = 0; c < NCH; ++c) {
+            const float4 a = q[c][r], b = k[c][r];
+            qq += (a.x * a.x + a.y * a.y) + (a.z * a.z + a.w * a.w);
+            kk += (b.x * b.x + b.y * b.y) + (b.z * b.z + b.w * b.w);
+            kq += (a.x * b.x + a.y * b.y) + (a.z * b.z + a.w * b.w);
+        }
+        const float fq = q_scale / sqrtf(warp_sum(qq) + 1e-6f), fk = 1.0f / sqrtf(warp_sum(kk) + 1e-6f);
+        const float dot = warp_sum(kq) * fq * fk;
+        if (r_first + r >= n_rows) continue;
+        float *o = conv + (size_t)(r_first + r) * ld;
+#pragma unroll
+        for (int c = 0; c < NCH; ++c) {
+            const int j = lane * 4 + 128 * c;
+            if (j < d.dim_p) {
+                const float4 a = q[c][r], b = k[c][r];
+                *reinterpret_cast<float4 *>(o + d.q_at() + u * d.dim_p + j) = make_float4(a.x * fq, a.y * fq, a.z * fq, a.w * fq);
+                *reinterpret_cast<float4 *>(o + d.k_at() + u * d.dim_p + j) = make_float4(b.x * fk, b.y * fk, b.z * fk, b.w * fk);
             }
         }
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const int row = r_first + 2 * half + r;
-            const float fq = q_scale / sqrtf(warp_sum(qq[r]) + 1e-6f), fk = 1.0f / sqrtf(warp_sum(kk[r]) + 1e-6f);
-            const float dot = warp_sum(kq[r]) * fq * fk;
-            if (row >= n_rows) continue;
-            float *o = conv + (size_t)row * ld;
-#pragma unroll
-            for (int c = 0; c < 2; ++c) {
-                const int j = lane * 4 + 128 * c;
-                if (j < d.dim_p) {
-                    const float4 a = q[r][c], b = k[r][c];
-                    *reinterpret_cast<float4 *>(o + d.q_at() + u * d.dim_p + j) = make_float4(a.x * fq, a.y * fq, a.z * fq, a.w * fq);
-                    *reinterpret_cast<float4 *>(o + d.k_at() + u * d.dim_p + j) = make_float4(b.x * fk, b.y * fk, b.z * fk, b.w * fk);
-                }
-            }
-            if (lane == 0) o[d.kq_at() + u] = dot;
-        }
+        if (lane == 0) o[d.kq_at() + u] = dot;
     }
 }
 
@@ -518,9 +541,13 @@ int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const flo
     if (d.dim_p > 256) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
     if (n_rows > 8 * 65535 || sm.n_seq > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: too many rows or sequences in a pass");
     if (ldp & 3) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: projection rows must keep 16-byte alignment");
-    PREFER_SMEM_ONCE(delta_conv_kernel);
-    launch_pdl(ctx, delta_conv_kernel, dim3(d.kv_heads + d.heads, (n_rows + 8 * CONV_ROWS - 1) / (8 * CONV_ROWS)), dim3(256), 0, d, proj, ldp, w,
-               conv_state, rows, sm, row_seq, n_rows, conv);
+    const dim3 cgrid(d.kv_heads + d.heads, (n_rows + 8 * CONV_ROWS - 1) / (8 * CONV_ROWS));
+    PREFER_SMEM_ONCE(delta_conv_kernel<1>);
+    PREFER_SMEM_ONCE(delta_conv_kernel<2>);
+    if (d.dim_p <= 128)
+        launch_pdl(ctx, delta_conv_kernel<1>, cgrid, dim3(256), 0, d, proj, ldp, w, conv_state, rows, sm, row_seq, n_rows, conv);
+    else
+        launch_pdl(ctx, delta_conv_kernel<2>, cgrid, dim3(256), 0, d, proj, ldp, w, conv_state, rows, sm, row_seq, n_rows, conv);
     CK_LAUNCH(ctx, "delta_conv_kernel");
     // columns per lane: two when that leaves every SM a dozen warps, else one (more parallel, more instructions)
     const long long columns = (long long)d.vdim_p * d.heads * sm.n_seq;

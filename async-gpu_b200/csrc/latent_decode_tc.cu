@@ -399,8 +399,11 @@ int tile_pairs_of(const LatentDims &d) { return (d.rank_p + 127) / 128; }
 size_t fixed_smem(const LatentDims &d, int n) { return 1024 + BOX + (size_t)((d.rank_p + 63) / 64 + 1) * n * 128 + (size_t)n * 256; }
 int ring_pairs_of(const LatentDims &d) {
     const int tp = tile_pairs_of(d);
-    const int fit = (int)((227 * 1024 - 2048 - fixed_smem(d, heads_per_block(d))) / PAIR);
-    return std::min({fit, 2 * tp, MAX_PAIRS});
+    const size_t fixed = fixed_smem(d, heads_per_block(d));
+    const int fit = (int)((227 * 1024 - 2048 - fixed) / PAIR);
+    // two blocks per SM where a tile fits in half of it (they cover each other's softmax), else one with the deepest ring
+    const int half = fixed + tp * PAIR <= 111 * 1024 ? (int)((111 * 1024 - fixed) / PAIR) : fit;
+    return std::min({fit, half, 2 * tp, MAX_PAIRS});
 }
 
 // Key splits per row: the number that minimises (waves of blocks) x (tiles per block + about one tile's worth of
@@ -409,7 +412,7 @@ int pick_splits(const b200nn_ctx *ctx, const LatentDims &d, int n_rows, int cap)
     const int n = heads_per_block(d), hb = (d.heads + n - 1) / n;
     const int tiles = ((d.window ? std::min(d.window + 127, cap) : cap) + 127) / 128;
     const size_t smem = fixed_smem(d, n) + (size_t)ring_pairs_of(d) * PAIR;
-    const long long per_wave = (long long)ctx->sm_count * std::max<size_t>(1, (227 * 1024) / (smem + 1024));
+    const long long per_wave = (long long)ctx->sm_count * std::max<size_t>(1, (227 * 1024) / (smem + 2048));
     int best = 1;
     double best_cost = 1e300;
     for (int s = 1; s <= std::min(tiles, 64); ++s) {
