@@ -319,7 +319,7 @@ __device__ __forceinline__ void cp_async4(void *smem, const void *gmem) {
 // Per token: both products against the old state, one reduction over the eight lanes (transposing: 2 NC values in
 // log steps), the write.  Also leaves the convolution's last inputs in the cache (blocks of column group 0).
 template <int DM, int NC>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, DM > 4 ? 1 : 5)
 delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ conv, float *__restrict__ conv_state,
                   float *__restrict__ state, SeqMap sm, float *__restrict__ heads_out) {
     constexpr int CH = DM <= 4 ? 16 : 8, DP = DM * 32, CB = 16 * NC;
@@ -351,17 +351,18 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
     auto copy = [&](int t0, Stage &st) {
         const int nt = min(CH, n - t0), dv = d.dim_p >> 2, cv = min(CB, d.vdim_p - cg * CB) >> 2;
         const float *c = conv + (size_t)(row0 + t0) * ldc;
-        for (int t = warp; t < nt; t += 4) { // a warp per token
-            const float *ct = c + (size_t)t * ldc;
-            for (int j = lane; j < dv; j += 32) {
-                cp_async16(&st.q[t][4 * j], ct + d.q_at() + kh * d.dim_p + 4 * j);
-                cp_async16(&st.k[t][4 * j], ct + d.k_at() + kh * d.dim_p + 4 * j);
-            }
-            if (lane < cv) cp_async16(&st.v[t][4 * lane], ct + d.v_at() + h * d.vdim_p + cg * CB + 4 * lane);
-            if (lane >= 29) {
-                const int j = lane - 29;
-                cp_async4(&st.s[t][j], ct + (j == 0 ? d.decay_at() + h : j == 1 ? d.beta_at() + h : d.kq_at() + kh));
-            }
+        for (int i = tid; i < nt * dv; i += 128) {
+            const int t = i / dv, j = (i - t * dv) * 4;
+            cp_async16(&st.q[t][j], c + (size_t)t * ldc + d.q_at() + kh * d.dim_p + j);
+            cp_async16(&st.k[t][j], c + (size_t)t * ldc + d.k_at() + kh * d.dim_p + j);
+        }
+        for (int i = tid; i < nt * cv; i += 128) {
+            const int t = i / cv, j = (i - t * cv) * 4;
+            cp_async16(&st.v[t][j], c + (size_t)t * ldc + d.v_at() + h * d.vdim_p + cg * CB + j);
+        }
+        for (int i = tid; i < nt * 3; i += 128) {
+            const int t = i / 3, j = i - t * 3;
+            cp_async4(&st.s[t][j], c + (size_t)t * ldc + (j == 0 ? d.decay_at() + h : j == 1 ? d.beta_at() + h : d.kq_at() + kh));
         }
     };
     __syncthreads();
@@ -382,6 +383,7 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
         __syncthreads();
         const Stage &st = stages[b];
         const int nt = min(CH, n - t0);
+#pragma unroll 1
         for (int t = 0; t < nt; ++t) {
             const float4 sc = *reinterpret_cast<const float4 *>(st.s[t]);
             G *= sc.x;
