@@ -319,7 +319,7 @@ __device__ __forceinline__ void cp_async4(void *smem, const void *gmem) {
 // Per token: both products against the old state, one reduction over the eight lanes (transposing: 2 NC values in
 // log steps), the write.  Also leaves the convolution's last inputs in the cache (blocks of column group 0).
 template <int DM, int NC>
-__global__ void __launch_bounds__(128, DM > 4 ? 1 : 5)
+__global__ void __launch_bounds__(128, DM > 4 ? 1 : 4)
 delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ conv, float *__restrict__ conv_state,
                   float *__restrict__ state, SeqMap sm, float *__restrict__ heads_out) {
     constexpr int CH = DM <= 4 ? 16 : 8, DP = DM * 32, CB = 16 * NC;
@@ -383,7 +383,7 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
         __syncthreads();
         const Stage &st = stages[b];
         const int nt = min(CH, n - t0);
-#pragma unroll 1
+#pragma unroll 4
         for (int t = 0; t < nt; ++t) {
             const float4 sc = *reinterpret_cast<const float4 *>(st.s[t]);
             G *= sc.x;
