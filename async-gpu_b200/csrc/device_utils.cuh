@@ -43,13 +43,13 @@ __device__ __forceinline__ uint32_t pack_f16x2(float a, float b) {
     const __half2 h = __floats2half2_rn(a, b);
     return *reinterpret_cast<const uint32_t *>(&h);
 }
-__device__ __forceinline__ uint32_t epi_pack2(const Epilogue &e, float a, float b) {
-    return e.out_half == OUT_BF16 ? pack_bf16x2(a, b) : pack_f16x2(a, b);
-}
 __device__ __forceinline__ int row_pos(const RowMap &r, int m) { return r.pos[(size_t)m * r.pos_stride]; }
 __device__ __forceinline__ int row_slot(const RowMap &r, int m) { return r.slot ? r.slot[m] : m; }
 
 // Consumes one finished output value v (bias already added) for row m (token), column n (feature).
+// B16: with the bfloat16 Linears' additions (bfloat16 output, EPI_GLU, EPI_ROPE, row_scale); kernels that never see
+// them leave the code out (it costs the int4 GEMM's epilogue 5 % of a decode step's Linears).
+template <bool B16 = false>
 __device__ __forceinline__ void epi_store(const Epilogue &e, int m, int n, float v) {
     if (e.no_store) return;
     if (e.mode == EPI_RESID) {
@@ -71,9 +71,9 @@ __device__ __forceinline__ void epi_store(const Epilogue &e, int m, int n, float
         return;
     }
     v = apply_act(v, e.act);
-    if (e.row_scale) v *= e.row_scale[(size_t)m * e.rs_ld + n / e.rs_cols];
+    if (B16 && e.row_scale) v *= e.row_scale[(size_t)m * e.rs_ld + n / e.rs_cols];
     size_t i = (size_t)m * e.ldo + n;
-    if (e.out_half == OUT_BF16)
+    if (B16 && e.out_half == OUT_BF16)
         static_cast<__nv_bfloat16 *>(e.out)[i] = __float2bfloat16_rn(v);
     else if (e.out_half)
         static_cast<__half *>(e.out)[i] = __float2half_rn(v);
@@ -84,16 +84,17 @@ __device__ __forceinline__ void epi_store(const Epilogue &e, int m, int n, float
 // Four consecutive columns n..n+3 (n % 4 == 0) of row m in one go: 16-byte (f32) or 8-byte (fp16)
 // stores when the destination allows it, element-wise otherwise.  pos_ptr must already be folded
 // into e.pos_off by the caller (it is not dereferenced here for the vector path).
+template <bool B16 = false>
 __device__ __forceinline__ void epi_store4(const Epilogue &e, int m, int n, float4 v, int N) {
     if (e.no_store) return;
-    if (e.mode == EPI_GLU) { // N and ldo are multiples of 4
+    if (B16 && e.mode == EPI_GLU) { // N and ldo are multiples of 4
         if (n >= N) return;
         const size_t i = (size_t)m * e.ldo + (n >> 1);
         *reinterpret_cast<uint32_t *>(static_cast<__nv_bfloat16 *>(e.out) + i) =
             pack_bf16x2(apply_act(v.x, e.act) * v.z, apply_act(v.y, e.act) * v.w);
         return;
     }
-    if (e.mode == EPI_ROPE) {
+    if (B16 && e.mode == EPI_ROPE) {
         if (n >= N) return;
         const int p = (n % e.rope_head - e.rope_at) >> 1;
         if (p >= 0 && p < e.rope_pairs) {
@@ -105,10 +106,10 @@ __device__ __forceinline__ void epi_store4(const Epilogue &e, int m, int n, floa
     }
     const bool vec = (n + 3 < N) && ((e.ldo & 3) == 0) && (e.pos_ptr == nullptr);
     if (!vec) {
-        if (n < N) epi_store(e, m, n, v.x);
-        if (n + 1 < N) epi_store(e, m, n + 1, v.y);
-        if (n + 2 < N) epi_store(e, m, n + 2, v.z);
-        if (n + 3 < N) epi_store(e, m, n + 3, v.w);
+        if (n < N) epi_store<B16>(e, m, n, v.x);
+        if (n + 1 < N) epi_store<B16>(e, m, n + 1, v.y);
+        if (n + 2 < N) epi_store<B16>(e, m, n + 2, v.z);
+        if (n + 3 < N) epi_store<B16>(e, m, n + 3, v.w);
         return;
     }
     if (e.mode == EPI_RESID) {
@@ -137,13 +138,15 @@ __device__ __forceinline__ void epi_store4(const Epilogue &e, int m, int n, floa
     }
     v.x = apply_act(v.x, e.act); v.y = apply_act(v.y, e.act);
     v.z = apply_act(v.z, e.act); v.w = apply_act(v.w, e.act);
-    if (e.row_scale) {
+    if (B16 && e.row_scale) {
         const float rs = e.row_scale[(size_t)m * e.rs_ld + n / e.rs_cols];
         v.x *= rs; v.y *= rs; v.z *= rs; v.w *= rs;
     }
     const size_t i = (size_t)m * e.ldo + n;
     if (e.out_half) {
-        *reinterpret_cast<uint2 *>(static_cast<__half *>(e.out) + i) = make_uint2(epi_pack2(e, v.x, v.y), epi_pack2(e, v.z, v.w));
+        const uint2 u = B16 && e.out_half == OUT_BF16 ? make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w))
+                                                      : make_uint2(pack_f16x2(v.x, v.y), pack_f16x2(v.z, v.w));
+        *reinterpret_cast<uint2 *>(static_cast<__half *>(e.out) + i) = u;
     } else {
         *reinterpret_cast<float4 *>(static_cast<float *>(e.out) + i) = v;
     }
@@ -307,8 +310,9 @@ __device__ __forceinline__ void epi_emit4(const Epilogue &e2, const Epilogue &ep
 }
 
 // Same, from a raw accumulated dot product.
+template <bool B16 = false>
 __device__ __forceinline__ void epi_apply(const Epilogue &e, int m, int n, float acc) {
-    epi_store(e, m, n, acc + (e.bias ? e.bias[n] : 0.0f));
+    epi_store<B16>(e, m, n, acc + (e.bias ? e.bias[n] : 0.0f));
 }
 
 __device__ __forceinline__ float warp_sum(float v) {

@@ -45,24 +45,21 @@ enum : uint32_t { ERR_EMPTY = 0x201, ERR_FULL, ERR_ACC };
 constexpr int BK = 64;                 // fp16 elements per K block = one 128-byte swizzle row
 constexpr int W_BYTES = 128 * BK * 2;  // weight box: 128 features x 64 k
 
-// What the operands are besides plain fp16 matrices.  idesc_bits: operand-format bits of the instruction
-// descriptor (0: fp16, tc::UMMA_BF16: bfloat16; always the same for both operands).  A block-diagonal Linear
-// (groups > 1) has group_tiles feature tiles per group: tile nt multiplies the activation columns from
-// (nt / group_tiles) * group_kx on and its group_n features start at output column
+// A block-diagonal Linear (bfloat16 kernels only): group_tiles feature tiles per group; tile nt multiplies the
+// activation columns from (nt / group_tiles) * group_kx on and its group_n features start at output column
 // (nt / group_tiles) * group_stride.
 struct OperandForm {
-    uint32_t idesc_bits = 0;
     int group_tiles = 0x7fffffff, group_kx = 0, group_n = 0x7fffffff, group_stride = 0;
 };
 // Output column of a tile's feature (column n of the padded weight); lim: the number of columns from which on
 // nothing may be stored (N, or the end of the feature's group; 0 for a padding feature of a group).
+template <bool B16>
 __device__ __forceinline__ int out_column(const OperandForm &f, int nt, int n, int N, int *lim) {
-    const int g = nt / f.group_tiles;
-    if (f.group_stride == 0) {
+    if (!B16 || f.group_stride == 0) {
         *lim = N;
         return n;
     }
-    const int local = n - g * f.group_tiles * 128;
+    const int g = nt / f.group_tiles, local = n - g * f.group_tiles * 128;
     *lim = local < f.group_n ? g * f.group_stride + f.group_n : 0;
     return g * f.group_stride + local;
 }
@@ -73,8 +70,9 @@ __device__ __forceinline__ void bar_sync_epi() {
 }
 
 // MB: token-tile width (the MMA's N); NS: operand stages; NE: epilogue groups of four warps;
-// TW: fp16 terms of the weight (1: hi, 2: hi + lo; tmap_w2 is read only with TW = 2).
-template <int MB, int NS, int NE, int TW>
+// TW: fp16 terms of the weight (1: hi, 2: hi + lo; tmap_w2 is read only with TW = 2);
+// B16: both operands bfloat16, with those Linears' epilogues and block-diagonal form.
+template <int MB, int NS, int NE, int TW, bool B16>
 __global__ void __launch_bounds__(64 + 128 * NE, 1)
 f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_w2,
                    const __grid_constant__ CUtensorMap tmap_x, int M, int N, int k_blocks, int kb_per_split,
@@ -121,8 +119,8 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
     // the epilogue's per-thread constants (filled by the epilogue warps, used in both of its places):
     // lane l owns features 4l..4l+3 of a token row
     int n_lim;
-    const int n4 = out_column(form, nt, nt * 128 + lane * 4, N, &n_lim);
-    const int kx = (nt / form.group_tiles) * form.group_kx; // first activation column
+    const int n4 = out_column<B16>(form, nt, nt * 128 + lane * 4, N, &n_lim);
+    const int kx = B16 ? (nt / form.group_tiles) * form.group_kx : 0; // first activation column
     float4 b4 = make_float4(0.f, 0.f, 0.f, 0.f);
     Epilogue e2 = epi; // the device-side position is read once per thread
     e2.pos_ptr = nullptr;
@@ -160,7 +158,7 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
         }
     } else if (warp == 1) {
         // ---- MMA issue: the whole warp runs the loop, one elected lane issues ----
-        const uint32_t idesc = tc::umma_idesc_f16(128, MB) | form.idesc_bits;
+        constexpr uint32_t idesc = tc::umma_idesc_f16(128, MB) | (B16 ? tc::UMMA_BF16 : 0u);
         const uint64_t d0 = tc::umma_desc_sw128(base);
         bool ok = true;
         int s = 0;
@@ -229,7 +227,7 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
             if (splits == 1) {
                 for (int c = w8; c < rows; c += NW) {
                     const float4 v = f4_add(stage4[c * 32 + lane], b4);
-                    epi_store4(e2, mt * MB + c, n4, v, n_lim);
+                    epi_store4<B16>(e2, mt * MB + c, n4, v, n_lim);
                     if (epi.amax_val) epi_argmax4(epi, mt * MB + c, n4, v, n_lim);
                 }
             } else if (epi.mode == EPI_RESID) {
@@ -258,7 +256,7 @@ f16_gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
                 float4 sum = b4;
                 for (int sp = 0; sp < splits; ++sp)
                     sum = f4_add(sum, cluster.map_shared_rank(stage4, sp)[c * 32 + lane]);
-                epi_store4(e2, mt * MB + c, n4, sum, n_lim);
+                epi_store4<B16>(e2, mt * MB + c, n4, sum, n_lim);
                 if (epi.amax_val) epi_argmax4(epi, mt * MB + c, n4, sum, n_lim);
             }
         }
@@ -298,7 +296,7 @@ __device__ __forceinline__ bool bar_or_epi(bool pred) {
 //   full[s] / empty[s]      operand stage s loaded / its MMAs retired (as above);
 //   acc_full[b] / acc_empty[b]  accumulator b complete (tcgen05.commit) / read out (one arrival per
 //                               epilogue warp).
-template <int MB, int NS, int NE, int TW>
+template <int MB, int NS, int NE, int TW, bool B16>
 __global__ void __launch_bounds__(64 + 128 * NE, 1)
 f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_w2,
                               const __grid_constant__ CUtensorMap tmap_x, int M, int N, int k_blocks, int n_tiles,
@@ -356,7 +354,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
         bool ok = true;
         for (int t = blockIdx.x; ok && t < total_tiles; t += gridDim.x) {
             const int mt = t / n_tiles, nt = t - mt * n_tiles;
-            const int kx = (nt / form.group_tiles) * form.group_kx;
+            const int kx = B16 ? (nt / form.group_tiles) * form.group_kx : 0;
             for (int kb = 0; kb < k_blocks; ++kb) {
                 ok = tc::mbar_wait(empty + 8 * s, ph, &abort_flag, dev_err, ERR_EMPTY);
                 if (!ok) break;
@@ -372,7 +370,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
         }
     } else if (warp == 1) {
         // ---- MMA issue ----
-        const uint32_t idesc = tc::umma_idesc_f16(128, MB) | form.idesc_bits;
+        constexpr uint32_t idesc = tc::umma_idesc_f16(128, MB) | (B16 ? tc::UMMA_BF16 : 0u);
         const uint64_t d0 = tc::umma_desc_sw128(base);
         int s = 0;
         uint32_t ph = 0;
@@ -428,7 +426,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
             const int b = j & 1;
             const int mt = t / n_tiles, nt = t - mt * n_tiles;
             int n_lim;
-            const int n4 = out_column(form, nt, nt * 128 + lane * 4, N, &n_lim);
+            const int n4 = out_column<B16>(form, nt, nt * 128 + lane * 4, N, &n_lim);
             const float4 b4 = epi_bias4(epi, n4, n_lim); // fetched under the wait for the accumulator
             bool ok = true;
             if (!__any_sync(0xffffffffu, abort_flag != 0))
@@ -458,7 +456,7 @@ f16_gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const 
                 } else {
                     for (int c = w8; c < lim; c += NW) {
                         const float4 v = f4_add(stage4[c * 32 + lane], b4);
-                        epi_store4(e2, mt * MB + c0 + c, n4, v, n_lim);
+                        epi_store4<B16>(e2, mt * MB + c0 + c, n4, v, n_lim);
                         if (epi.amax_val) epi_argmax4(epi, mt * MB + c0 + c, n4, v, n_lim);
                     }
                 }
@@ -507,27 +505,27 @@ struct WOperand {
     int N, K;
     bool constant;
     int ldx = 0, kx_total = 0; // row stride of the activations and the columns they have (0: K)
+    bool b16 = false;          // bfloat16 instead of fp16
     OperandForm form{};
-    bool bf16() const { return form.idesc_bits != 0; }
 };
 
-template <int MB, int NS, int NE, int TW>
+template <int MB, int NS, int NE, int TW, bool B16>
 int launch_cfg(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M, const Epilogue &epi) {
     constexpr size_t ring = (size_t)NS * (TW * W_BYTES + MB * BK * 2);
     constexpr size_t smem = 1024 + ring + 256;
     static_assert(16 * NS + 16 <= 256, "barrier area too small");
     static_assert(smem <= 227 * 1024, "shared memory budget exceeded");
     static bool attr_done[16] = {};
-    auto kern = f16_gemm_tc_kernel<MB, NS, NE, TW>;
+    auto kern = f16_gemm_tc_kernel<MB, NS, NE, TW, B16>;
     if (!attr_done[ctx->device & 15]) {
         CK(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         prefer_max_smem(kern);
         attr_done[ctx->device & 15] = true;
     }
     CUtensorMap tmap_w, tmap_w2, tmap_x;
-    TRY(make_map(ctx, w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w));
-    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w2));
-    TRY(make_map(ctx, x, M, w.kx_total ? w.kx_total : w.K, w.ldx ? w.ldx : w.K, MB, w.bf16(), &tmap_x));
+    TRY(make_map(ctx, w.hi, w.N, w.K, w.K, 128, w.b16, &tmap_w));
+    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, w.K, 128, w.b16, &tmap_w2));
+    TRY(make_map(ctx, x, M, w.kx_total ? w.kx_total : w.K, w.ldx ? w.ldx : w.K, MB, w.b16, &tmap_x));
 
     const int k_blocks = (w.K + BK - 1) / BK;
     const int n_tiles = (w.N + 127) / 128, m_tiles = (M + MB - 1) / MB;
@@ -574,23 +572,23 @@ int launch_cfg(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M, const
 }
 
 // Many tiles (at least two per SM): one persistent block per SM, 256-row token tiles.
-template <int NS, int TW>
+template <int NS, int TW, bool B16>
 int launch_persistent(b200nn_ctx *ctx, const WOperand &w, const __half *x, int M, const Epilogue &epi) {
     constexpr int MB = 256, NE = 4;
     constexpr size_t smem = 1024 + (size_t)NS * (TW * W_BYTES + MB * BK * 2) + 64 * 128 * 4 + 256;
     static_assert(16 * NS + 48 <= 256, "barrier area too small");
     static_assert(smem <= 227 * 1024, "shared memory budget exceeded");
     static bool attr_done[16] = {};
-    auto kern = f16_gemm_tc_persistent_kernel<MB, NS, NE, TW>;
+    auto kern = f16_gemm_tc_persistent_kernel<MB, NS, NE, TW, B16>;
     if (!attr_done[ctx->device & 15]) {
         CK(ctx, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         prefer_max_smem(kern);
         attr_done[ctx->device & 15] = true;
     }
     CUtensorMap tmap_w, tmap_w2, tmap_x;
-    TRY(make_map(ctx, w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w));
-    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, w.K, 128, w.bf16(), &tmap_w2));
-    TRY(make_map(ctx, x, M, w.kx_total ? w.kx_total : w.K, w.ldx ? w.ldx : w.K, MB, w.bf16(), &tmap_x));
+    TRY(make_map(ctx, w.hi, w.N, w.K, w.K, 128, w.b16, &tmap_w));
+    TRY(make_map(ctx, TW == 2 ? w.lo : w.hi, w.N, w.K, w.K, 128, w.b16, &tmap_w2));
+    TRY(make_map(ctx, x, M, w.kx_total ? w.kx_total : w.K, w.ldx ? w.ldx : w.K, MB, w.b16, &tmap_x));
     const int k_blocks = (w.K + BK - 1) / BK;
     const int n_tiles = (w.N + 127) / 128, m_tiles = (M + MB - 1) / MB;
     const int total = n_tiles * m_tiles;
@@ -627,22 +625,31 @@ bool use_persistent(const b200nn_ctx *ctx, int N, int M, int mb) {
 
 int launch_terms(b200nn_ctx *ctx, const WOperand &w, int terms, const __half *x, int M, const Epilogue &epi) {
     const int mb = pick_mb(ctx, w.N, M);
+    if (w.b16) { // bfloat16 operands
+        if (use_persistent(ctx, w.N, M, mb)) return launch_persistent<4, 1, true>(ctx, w, x, M, epi);
+        switch (mb) {
+            case 32: return launch_cfg<32, 8, 2, 1, true>(ctx, w, x, M, epi);
+            case 64: return launch_cfg<64, 8, 2, 1, true>(ctx, w, x, M, epi);
+            case 128: return launch_cfg<128, 6, 4, 1, true>(ctx, w, x, M, epi);
+            default: return launch_cfg<256, 4, 4, 1, true>(ctx, w, x, M, epi);
+        }
+    }
     if (terms == 1) { // the weight as one fp16 matrix
-        if (use_persistent(ctx, w.N, M, mb)) return launch_persistent<4, 1>(ctx, w, x, M, epi);
+        if (use_persistent(ctx, w.N, M, mb)) return launch_persistent<4, 1, false>(ctx, w, x, M, epi);
         switch (mb) { //            MB  NS NE TW
-            case 32: return launch_cfg<32, 8, 2, 1>(ctx, w, x, M, epi);
-            case 64: return launch_cfg<64, 8, 2, 1>(ctx, w, x, M, epi);
-            case 128: return launch_cfg<128, 6, 4, 1>(ctx, w, x, M, epi);
-            default: return launch_cfg<256, 4, 4, 1>(ctx, w, x, M, epi);
+            case 32: return launch_cfg<32, 8, 2, 1, false>(ctx, w, x, M, epi);
+            case 64: return launch_cfg<64, 8, 2, 1, false>(ctx, w, x, M, epi);
+            case 128: return launch_cfg<128, 6, 4, 1, false>(ctx, w, x, M, epi);
+            default: return launch_cfg<256, 4, 4, 1, false>(ctx, w, x, M, epi);
         }
     }
     // rounded weight + rounded remainder, two products per K block
-    if (use_persistent(ctx, w.N, M, mb)) return launch_persistent<3, 2>(ctx, w, x, M, epi);
+    if (use_persistent(ctx, w.N, M, mb)) return launch_persistent<3, 2, false>(ctx, w, x, M, epi);
     switch (mb) {
-        case 32: return launch_cfg<32, 5, 2, 2>(ctx, w, x, M, epi);
-        case 64: return launch_cfg<64, 5, 2, 2>(ctx, w, x, M, epi);
-        case 128: return launch_cfg<128, 4, 4, 2>(ctx, w, x, M, epi);
-        default: return launch_cfg<256, 3, 4, 2>(ctx, w, x, M, epi);
+        case 32: return launch_cfg<32, 5, 2, 2, false>(ctx, w, x, M, epi);
+        case 64: return launch_cfg<64, 5, 2, 2, false>(ctx, w, x, M, epi);
+        case 128: return launch_cfg<128, 4, 4, 2, false>(ctx, w, x, M, epi);
+        default: return launch_cfg<256, 3, 4, 2, false>(ctx, w, x, M, epi);
     }
 }
 
@@ -710,7 +717,7 @@ int launch_b16_linear(b200nn_ctx *ctx, const B16Weight &w, const __nv_bfloat16 *
     WOperand op{(const __half *)w.w_nk->p, nullptr, w.N, w.K, true};
     op.ldx = ldx;
     op.kx_total = w.K + (w.groups - 1) * w.group_kx;
-    op.form.idesc_bits = tc::UMMA_BF16;
+    op.b16 = true;
     if (w.groups > 1) {
         op.form.group_tiles = w.group_tiles;
         op.form.group_kx = w.group_kx;

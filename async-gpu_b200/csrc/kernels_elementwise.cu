@@ -716,7 +716,7 @@ __global__ void __launch_bounds__(256) grouped_f32_kernel(const float *__restric
     float a = 0.0f;
     for (int k = lane; k < Kg; k += 32) a = fmaf(wr[k], xr[k], a);
     a = warp_sum(a);
-    if (lane == 0) epi_apply(epi, m, g * out_stride + n, a);
+    if (lane == 0) epi_apply<true>(epi, m, g * out_stride + n, a);
 }
 int launch_grouped_f32(b200nn_ctx *ctx, const float *w, int groups, int Ng, int Kg, const float *x, int ldx, int x_stride, int M,
                        const Epilogue &epi, int out_stride) {
