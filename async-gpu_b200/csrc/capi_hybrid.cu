@@ -76,7 +76,7 @@ extern "C" int32_t b200nn_delta_rule(b200nn_ctx *ctx, const b200nn_delta_shape *
     const DeltaWeights dw{w->conv, w->a_exp, w->dt_bias, w->norm};
     const bool b16 = !(flags & B200NN_LM_F32);
     const RowMap rows{pos_dev, 1, slot_dev};
-    if (n_seq == 0) return launch_delta_step(ctx, d, b16, proj_dev, d.proj_w(), dw, conv_state_dev, state_dev, rows, n_rows, out_dev);
+    if (n_seq == 0) return launch_delta_step(ctx, d, b16, proj_dev, d.proj_w(), nullptr, dw, conv_state_dev, state_dev, rows, n_rows, out_dev);
     if (!seq_dev || !slot_dev || max_n <= 0 || unaligned({scratch_dev})) return B200NN_ERR_ARG;
     SeqMap sm;
     sm.n_seq = n_seq;
@@ -85,6 +85,6 @@ extern "C" int32_t b200nn_delta_rule(b200nn_ctx *ctx, const b200nn_delta_shape *
     sm.row0 = seq_dev + n_seq;
     sm.n = seq_dev + 2 * n_seq;
     sm.past = seq_dev + 3 * n_seq;
-    return launch_delta_prompt(ctx, d, b16, proj_dev, d.proj_w(), dw, conv_state_dev, state_dev, rows, sm, n_rows, seq_dev + 4 * n_seq, scratch_dev,
+    return launch_delta_prompt(ctx, d, b16, proj_dev, d.proj_w(), nullptr, dw, conv_state_dev, state_dev, rows, sm, n_rows, seq_dev + 4 * n_seq, scratch_dev,
                                scratch_dev + (size_t)n_rows * d.conv_ld(), out_dev);
 }

@@ -293,6 +293,14 @@ struct Epilogue {
     // row_scale: finished values are multiplied by row_scale[m * rs_ld + n / rs_cols] (a per-head gate)
     const float *row_scale = nullptr;
     int rs_ld = 0, rs_cols = 1;
+    // A Linear of several parts (bfloat16 Linears; both bounds multiples of 4): features from tail_at on go to
+    // tail_out [m][tail_ld] in an element type of their own; features kv_at .. tail_at are a key / value cache row,
+    // kv_w per head, stored at [slot][head][position][kv_w] of a bfloat16 cache of kv_heads heads and kv_cap
+    // positions (slot and position from rows).
+    void *tail_out = nullptr;
+    int tail_at = 0, tail_ld = 0, tail_type = OUT_F32;
+    __nv_bfloat16 *kv_cache = nullptr;
+    int kv_at = 0, kv_w = 0, kv_heads = 0, kv_cap = 0;
 };
 
 // ---------------------------------------------------------------------------------------------

@@ -3,6 +3,9 @@
 // taken on the state before the write: S_new^T q = g S^T q + (k . q) u, so a token costs one pass over the
 // state and one reduction instead of two.  Everything here is f32.
 //
+// The decay g is one number per head, or (CH, DeltaDims::channel) one per head and key channel, acting on the rows of
+// S; the output gate is then a sigmoid and its input, like the decays', comes from a projection of its own (`ext`).
+//
 //   delta_step_kernel     decoding: convolution, norms, recurrence, output norm and gate of one token
 //   delta_conv_kernel     prompts: convolution + silu, unit norms, k . q, decay and step size of every row
 //   delta_scan_kernel     prompts: the recurrence (state columns are independent: a block owns some of them)
@@ -20,7 +23,6 @@ namespace {
 // activation of the convolution and of the output gate (not part of the recurrence): fast exponential and division
 __device__ __forceinline__ float silu_f(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
 __device__ __forceinline__ float softplus_f(float v) { return v > 20.0f ? v : log1pf(expf(v)); }
-__device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
 __device__ __forceinline__ float decay_f(float a_exp, float a, float dt_bias) { return expf(-a_exp * softplus_f(a + dt_bias)); }
 
 // ---- decoding ----------------------------------------------------------------------------------------
@@ -28,13 +30,15 @@ __device__ __forceinline__ float decay_f(float a_exp, float a, float dt_bias) { 
 // 128-column chunk (one chunk for vdim <= 128).  Under the state's loads warps 0, 1 and 2 make the query, key and value
 // (a lane takes four channels; the unit norms stay scalar factors), warp 3 gate times norm weight, warp 4 decay and
 // step size.
-template <int RPW, typename T>
+template <int RPW, bool CH, typename T>
 __global__ void __launch_bounds__(256, RPW <= 16 ? 2 : 1)
-delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWeights w, float *__restrict__ conv_state,
+delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ ext, DeltaWeights w, float *__restrict__ conv_state,
                   float *__restrict__ state, RowMap rows, T *__restrict__ out) {
-    extern __shared__ __align__(16) float sh[]; // q [dim_p], k [dim_p], v, gate, o [vdim_p], reduction [8][2][128], scalars [8]
+    // q [dim_p], k [dim_p], v, gate, o [vdim_p], reduction [8][2][128], scalars [8], CH: decays [dim_p]
+    extern __shared__ __align__(16) float sh[];
     const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     float *sq = sh, *sk = sq + d.dim_p, *sv = sk + d.dim_p, *sgn = sv + d.vdim_p, *so = sgn + d.vdim_p, *red = so + d.vdim_p, *sc = red + 2048;
+    float *sg = sc + 8;
     pdl_trigger();
     pdl_wait();
     const int pos = row_pos(rows, row), slot = row_slot(rows, row);
@@ -101,17 +105,23 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         if (lane == 0) sc[2 + warp] = 1.0f / sqrtf(s + 1e-6f); // unit norms (the value's is not used)
     } else if (warp == 3) {
         for (int j = lane * 4; j < d.vdim_p; j += 128) { // the last columns may be padding: no norm weight there
-            const float4 gg = *reinterpret_cast<const float4 *>(p + d.g_at() + h * d.vdim_p + j);
+            const float *gate = CH ? ext + (size_t)row * 2 * d.ext() + d.ext() : p + d.g_at();
+            const float4 gg = *reinterpret_cast<const float4 *>(gate + h * d.vdim_p + j);
             const float e[4] = {gg.x, gg.y, gg.z, gg.w};
 #pragma unroll
-            for (int i = 0; i < 4; ++i) sgn[j + i] = j + i < d.vdim ? w.norm[j + i] * silu_f(e[i]) : 0.0f;
+            for (int i = 0; i < 4; ++i) sgn[j + i] = j + i < d.vdim ? w.norm[j + i] * (CH ? sigmoid_f(e[i]) : silu_f(e[i])) : 0.0f;
         }
-    } else if (tid == 128) {
+    } else if (CH && warp == 4) {
+        if (lane == 0) sc[0] = sigmoid_f(p[d.b_at() + h]);
+        const float a_exp = w.a_exp[h];
+        for (int j = lane; j < d.dim_p; j += 32)
+            sg[j] = decay_f(a_exp, ext[(size_t)row * 2 * d.ext() + h * d.dim_p + j], w.dt_bias[h * d.dim_p + j]);
+    } else if (!CH && tid == 128) {
         sc[0] = sigmoid_f(p[d.b_at() + h]);
         sc[1] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
     }
     __syncthreads();
-    const float beta = sc[0], g = sc[1], fq = sc[2] / sqrtf((float)d.dim), fk = sc[3]; // q also times dim^(-1/2)
+    const float beta = sc[0], g = CH ? 1.0f : sc[1], fq = sc[2] / sqrtf((float)d.dim), fk = sc[3]; // q also times dim^(-1/2)
     float kq = 0.0f; // warp 0, which makes the read-out, needs k . q
     if (warp == 0) {
         for (int j = lane; j < d.dim_p; j += 32) kq = fmaf(sk[j], sq[j], kq);
@@ -124,7 +134,7 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         for (int r = 0; r < RPW; ++r) {
             const int i = warp + 8 * r;
             if (i < d.dim_p) {
-                const float k = sk[i], q = sq[i];
+                const float gi = CH ? sg[i] : 1.0f, k = CH ? gi * sk[i] : sk[i], q = CH ? gi * sq[i] : sq[i];
                 ak.x = fmaf(st[r].x, k, ak.x); ak.y = fmaf(st[r].y, k, ak.y); ak.z = fmaf(st[r].z, k, ak.z); ak.w = fmaf(st[r].w, k, ak.w);
                 aq.x = fmaf(st[r].x, q, aq.x); aq.y = fmaf(st[r].y, q, aq.y); aq.z = fmaf(st[r].z, q, aq.z); aq.w = fmaf(st[r].w, q, aq.w);
             }
@@ -147,9 +157,9 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
             for (int r = 0; r < RPW; ++r) {
                 const int i = warp + 8 * r;
                 if (i < d.dim_p) {
-                    const float k = sk[i] * fk;
+                    const float k = sk[i] * fk, gi = CH ? sg[i] : g;
                     *reinterpret_cast<float4 *>(S + (size_t)i * d.vdim_p + c) =
-                        make_float4(fmaf(k, u.x, g * st[r].x), fmaf(k, u.y, g * st[r].y), fmaf(k, u.z, g * st[r].z), fmaf(k, u.w, g * st[r].w));
+                        make_float4(fmaf(k, u.x, gi * st[r].x), fmaf(k, u.y, gi * st[r].y), fmaf(k, u.z, gi * st[r].z), fmaf(k, u.w, gi * st[r].w));
                 }
             }
             if (warp == 0)
@@ -174,9 +184,9 @@ delta_step_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
 // block take neighbouring rows, which share their convolution inputs in L1.
 // NCH: 128-channel chunks of a query/key head.
 constexpr int CONV_ROWS = 4;
-template <int NCH>
+template <int NCH, bool CH>
 __global__ void __launch_bounds__(256)
-delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWeights w, const float *__restrict__ conv_state, RowMap rows,
+delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ ext, DeltaWeights w, const float *__restrict__ conv_state, RowMap rows,
                   SeqMap sm, const int *__restrict__ row_seq, int n_rows, float *__restrict__ conv) {
     pdl_trigger();
     pdl_wait();
@@ -240,8 +250,21 @@ delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
         if (lane < CONV_ROWS && r_first + lane < n_rows) {
             const float *p = proj + (size_t)(r_first + lane) * ldp;
             float *o = conv + (size_t)(r_first + lane) * ld;
-            o[d.decay_at() + h] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
+            if (!CH) o[d.decay_at() + h] = decay_f(w.a_exp[h], p[d.a_at() + h], w.dt_bias[h]);
             o[d.beta_at() + h] = sigmoid_f(p[d.b_at() + h]);
+        }
+        if (CH) {
+            const float a_exp = w.a_exp[h];
+            for (int j = lane * 4; j < d.dim_p; j += 128) {
+                const float4 b = __ldg(reinterpret_cast<const float4 *>(w.dt_bias + h * d.dim_p + j));
+#pragma unroll
+                for (int r = 0; r < CONV_ROWS; ++r) {
+                    if (r_first + r >= n_rows) break;
+                    const float4 a = *reinterpret_cast<const float4 *>(ext + (size_t)(r_first + r) * 2 * d.ext() + h * d.dim_p + j);
+                    *reinterpret_cast<float4 *>(conv + (size_t)(r_first + r) * ld + d.decay_at() + h * d.dim_p + j) =
+                        make_float4(decay_f(a_exp, a.x, b.x), decay_f(a_exp, a.y, b.y), decay_f(a_exp, a.z, b.z), decay_f(a_exp, a.w, b.w));
+                }
+            }
         }
         return;
     }
@@ -284,47 +307,20 @@ delta_conv_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, DeltaWei
     }
 }
 
-// Pairs of f32 in one register pair: one instruction for two multiply-adds.
-__device__ __forceinline__ uint64_t f32x2(float a, float b) {
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-    return r;
-}
-__device__ __forceinline__ float2 f32x2_parts(uint64_t v) {
-    float2 r;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
-    return r;
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t r;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-    return r;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-    uint64_t r;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-    return r;
-}
-__device__ __forceinline__ void cp_async16(void *smem, const void *gmem) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
-}
-__device__ __forceinline__ void cp_async4(void *smem, const void *gmem) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
-}
-
 // Block = (16 NC state columns, head, sequence), four warps.  The eight lanes of a column group hold its dim entries
-// 4 l + 32 m .. + 3 of NC columns each (f32 pairs along dim).  Tokens come through shared memory CH at a time, the next
-// CH being copied under the current ones.  The state is held divided by the decay G accumulated since it was last
+// 4 l + 32 m .. + 3 of NC columns each (f32 pairs along dim).  Tokens come through shared memory TOK at a time, the next
+// TOK being copied under the current ones.  The state is held divided by the decay G accumulated since it was last
 // rescaled (S = G s), so that a token costs three multiply-adds per entry; it is rescaled when G falls below 2^-20.
+// With CH the decays differ along dim and are multiplied in directly (one multiply more per entry).
 // Per token: both products against the old state, one reduction over the eight lanes (transposing: 2 NC values in
 // log steps), the write.  Also leaves the convolution's last inputs in the cache (blocks of column group 0).
-template <int DM, int NC>
+template <int DM, int NC, bool CH>
 __global__ void __launch_bounds__(128, DM > 4 ? 1 : 4)
 delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ conv, float *__restrict__ conv_state,
                   float *__restrict__ state, SeqMap sm, float *__restrict__ heads_out) {
-    constexpr int CH = DM <= 4 ? 16 : 8, DP = DM * 32, CB = 16 * NC;
+    constexpr int TOK = DM <= 4 ? 16 : 8, DP = DM * 32, CB = 16 * NC;
     struct Stage {
-        float k[CH][DP], q[CH][DP], v[CH][CB], s[CH][4]; // s: decay, step size, k . q
+        float k[TOK][DP], q[TOK][DP], v[TOK][CB], s[TOK][4], g[CH ? TOK : 1][CH ? DP : 4]; // s: decay, step size, k . q; g: decays
     };
     extern __shared__ __align__(16) uint8_t smem_raw[];
     Stage *stages = reinterpret_cast<Stage *>(smem_raw);
@@ -349,12 +345,13 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
             }
         }
     auto copy = [&](int t0, Stage &st) {
-        const int nt = min(CH, n - t0), dv = d.dim_p >> 2, cv = min(CB, d.vdim_p - cg * CB) >> 2;
+        const int nt = min(TOK, n - t0), dv = d.dim_p >> 2, cv = min(CB, d.vdim_p - cg * CB) >> 2;
         const float *c = conv + (size_t)(row0 + t0) * ldc;
         for (int i = tid; i < nt * dv; i += 128) {
             const int t = i / dv, j = (i - t * dv) * 4;
             cp_async16(&st.q[t][j], c + (size_t)t * ldc + d.q_at() + kh * d.dim_p + j);
             cp_async16(&st.k[t][j], c + (size_t)t * ldc + d.k_at() + kh * d.dim_p + j);
+            if constexpr (CH) cp_async16(&st.g[t][j], c + (size_t)t * ldc + d.decay_at() + h * d.dim_p + j);
         }
         for (int i = tid; i < nt * cv; i += 128) {
             const int t = i / cv, j = (i - t * cv) * 4;
@@ -362,6 +359,7 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
         }
         for (int i = tid; i < nt * 3; i += 128) {
             const int t = i / 3, j = i - t * 3;
+            if (CH && j == 0) continue;
             cp_async4(&st.s[t][j], c + (size_t)t * ldc + (j == 0 ? d.decay_at() + h : j == 1 ? d.beta_at() + h : d.kq_at() + kh));
         }
     };
@@ -376,20 +374,32 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
 #pragma unroll
             for (int m = 0; m < DM * 2; ++m) s[c][m] = mul2(f2, s[c][m]);
     };
-    for (int t0 = 0, b = 0; t0 < n; t0 += CH, b ^= 1) {
-        if (t0 + CH < n) copy(t0 + CH, stages[b ^ 1]);
+    for (int t0 = 0, b = 0; t0 < n; t0 += TOK, b ^= 1) {
+        if (t0 + TOK < n) copy(t0 + TOK, stages[b ^ 1]);
         asm volatile("cp.async.commit_group;" ::: "memory");
         asm volatile("cp.async.wait_group 1;" ::: "memory");
         __syncthreads();
         const Stage &st = stages[b];
-        const int nt = min(CH, n - t0);
+        const int nt = min(TOK, n - t0);
 #pragma unroll 4
         for (int t = 0; t < nt; ++t) {
             const float4 sc = *reinterpret_cast<const float4 *>(st.s[t]);
-            G *= sc.x;
-            if (G < 9.5367431640625e-7f) { // the same in every thread of the block
-                rescale(G);
-                G = 1.0f;
+            if constexpr (CH) {
+#pragma unroll
+                for (int m = 0; m < DM; ++m) {
+                    const ulonglong2 gg = *reinterpret_cast<const ulonglong2 *>(&st.g[t][32 * m + 4 * part]);
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        s[c][2 * m] = mul2(gg.x, s[c][2 * m]);
+                        s[c][2 * m + 1] = mul2(gg.y, s[c][2 * m + 1]);
+                    }
+                }
+            } else {
+                G *= sc.x;
+                if (G < 9.5367431640625e-7f) { // the same in every thread of the block
+                    rescale(G);
+                    G = 1.0f;
+                }
             }
             uint64_t k[DM * 2];
             float r[2 * NC]; // s^T k of the NC columns, then s^T q
@@ -432,11 +442,11 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
             for (; o; o >>= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], o);
             // lanes with bit 4 clear now hold s^T k, the others s^T q, of column idx
             const int idx = NC == 1 ? 0 : (lane >> 1) & 1;
-            const float mine = G * r[0], other = __shfl_xor_sync(0xffffffffu, mine, 4);
+            const float mine = CH ? r[0] : G * r[0], other = __shfl_xor_sync(0xffffffffu, mine, 4);
             const float u_own = sc.y * (st.v[t][cl + idx] - ((lane & 4) ? other : mine));
             if ((lane & 4) && !(lane & 1) && (NC == 2 || !(lane & 2)) && col + idx < d.vdim_p)
                 heads_out[((size_t)(row0 + t0 + t) * d.heads + h) * d.vdim_p + col + idx] = fmaf(sc.z, u_own, mine);
-            const float us = __fdividef(u_own, G);
+            const float us = CH ? u_own : __fdividef(u_own, G);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 const float u = NC == 1 ? us : __shfl_sync(0xffffffffu, us, (lane & 24) | (c << 1));
@@ -447,7 +457,7 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
         }
         __syncthreads();
     }
-    rescale(G);
+    if (!CH) rescale(G);
 #pragma unroll
     for (int m = 0; m < DM; ++m)
 #pragma unroll
@@ -477,16 +487,17 @@ delta_scan_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const fl
 }
 
 // One warp per (row, head).
-template <typename T>
+template <bool CH, typename T>
 __global__ void __launch_bounds__(256)
-delta_out_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const float *__restrict__ norm, const float *__restrict__ heads_out,
+delta_out_kernel(DeltaDims d, const float *__restrict__ gates, int ldg, const float *__restrict__ norm, const float *__restrict__ heads_out,
                  int n_rows, T *__restrict__ out) {
     pdl_trigger();
     pdl_wait();
     const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (unit >= n_rows * d.heads) return;
     const int row = unit / d.heads, h = unit - row * d.heads;
-    const float *o = heads_out + (size_t)unit * d.vdim_p, *g = proj + (size_t)row * ldp + d.g_at() + h * d.vdim_p;
+    const float *o = heads_out + (size_t)unit * d.vdim_p, *g = gates + (size_t)row * ldg + h * d.vdim_p;
+    auto act = [](float z) { return CH ? sigmoid_f(z) : silu_f(z); };
     float4 v[2]; // the first 256 columns stay in registers
     float s = 0.0f;
 #pragma unroll
@@ -503,53 +514,42 @@ delta_out_kernel(DeltaDims d, const float *__restrict__ proj, int ldp, const flo
         const int j = lane * 4 + 128 * c;
         if (j >= d.vdim_p) continue;
         const float4 gg = __ldcs(reinterpret_cast<const float4 *>(g + j));
-        const float e[4] = {v[c].x * silu_f(gg.x), v[c].y * silu_f(gg.y), v[c].z * silu_f(gg.z), v[c].w * silu_f(gg.w)};
+        const float e[4] = {v[c].x * act(gg.x), v[c].y * act(gg.y), v[c].z * act(gg.z), v[c].w * act(gg.w)};
 #pragma unroll
         for (int i = 0; i < 4; ++i) store_from_float(y + j + i, j + i < d.vdim ? e[i] * rn * norm[j + i] : 0.0f);
     }
-    for (int j = 256 + lane; j < d.vdim; j += 32) store_from_float(y + j, o[j] * rn * norm[j] * silu_f(g[j]));
+    for (int j = 256 + lane; j < d.vdim; j += 32) store_from_float(y + j, o[j] * rn * norm[j] * act(g[j]));
 }
 
-}  // namespace
-
-int launch_delta_step(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const DeltaWeights &w, float *conv_state,
-                      float *state, const RowMap &rows, int n_rows, void *out) {
-    if (n_rows > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: more than 65535 rows");
+template <bool CH, typename T>
+int step_launch(b200nn_ctx *ctx, const DeltaDims &d, const float *proj, int ldp, const float *ext, const DeltaWeights &w, float *conv_state, float *state,
+                const RowMap &rows, int n_rows, T *out) {
     const dim3 grid(d.heads, n_rows);
-    const size_t smem = (2 * d.dim_p + 3 * d.vdim_p + 2048 + 8) * sizeof(float);
+    const size_t smem = (2 * d.dim_p + 3 * d.vdim_p + 2048 + 8 + (CH ? d.dim_p : 0)) * sizeof(float);
 #define DSTEP(R)                                                                                                             \
     do {                                                                                                                     \
-        PREFER_SMEM_ONCE((delta_step_kernel<R, __nv_bfloat16>));                                                             \
-        PREFER_SMEM_ONCE((delta_step_kernel<R, float>));                                                                     \
-        if (b16)                                                                                                             \
-            launch_pdl(ctx, delta_step_kernel<R, __nv_bfloat16>, grid, dim3(256), smem, d, proj, ldp, w, conv_state, state,  \
-                       rows, (__nv_bfloat16 *)out);                                                                          \
-        else                                                                                                                 \
-            launch_pdl(ctx, delta_step_kernel<R, float>, grid, dim3(256), smem, d, proj, ldp, w, conv_state, state, rows,    \
-                       (float *)out);                                                                                        \
+        PREFER_SMEM_ONCE((delta_step_kernel<R, CH, T>));                                                                     \
+        launch_pdl(ctx, delta_step_kernel<R, CH, T>, grid, dim3(256), smem, d, proj, ldp, ext, w, conv_state, state, rows,   \
+                   out);                                                                                                     \
     } while (0)
     if (d.dim_p <= 64) DSTEP(8);
     else if (d.dim_p <= 128) DSTEP(16);
-    else if (d.dim_p <= 256) DSTEP(32);
-    else return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
+    else DSTEP(32);
 #undef DSTEP
     CK_LAUNCH(ctx, "delta_step_kernel");
     return B200NN_OK;
 }
 
-int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const DeltaWeights &w,
-                        float *conv_state, float *state, const RowMap &rows, const SeqMap &sm, int n_rows, const int *row_seq, float *conv,
-                        float *heads_out, void *out) {
-    if (d.dim_p > 256) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
-    if (n_rows > 8 * 65535 || sm.n_seq > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: too many rows or sequences in a pass");
-    if (ldp & 3) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: projection rows must keep 16-byte alignment");
+template <bool CH>
+int prompt_launch(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const float *ext, const DeltaWeights &w, float *conv_state,
+                  float *state, const RowMap &rows, const SeqMap &sm, int n_rows, const int *row_seq, float *conv, float *heads_out, void *out) {
     const dim3 cgrid(d.kv_heads + d.heads, (n_rows + 8 * CONV_ROWS - 1) / (8 * CONV_ROWS));
-    PREFER_SMEM_ONCE(delta_conv_kernel<1>);
-    PREFER_SMEM_ONCE(delta_conv_kernel<2>);
+    PREFER_SMEM_ONCE((delta_conv_kernel<1, CH>));
+    PREFER_SMEM_ONCE((delta_conv_kernel<2, CH>));
     if (d.dim_p <= 128)
-        launch_pdl(ctx, delta_conv_kernel<1>, cgrid, dim3(256), 0, d, proj, ldp, w, conv_state, rows, sm, row_seq, n_rows, conv);
+        launch_pdl(ctx, delta_conv_kernel<1, CH>, cgrid, dim3(256), 0, d, proj, ldp, ext, w, conv_state, rows, sm, row_seq, n_rows, conv);
     else
-        launch_pdl(ctx, delta_conv_kernel<2>, cgrid, dim3(256), 0, d, proj, ldp, w, conv_state, rows, sm, row_seq, n_rows, conv);
+        launch_pdl(ctx, delta_conv_kernel<2, CH>, cgrid, dim3(256), 0, d, proj, ldp, ext, w, conv_state, rows, sm, row_seq, n_rows, conv);
     CK_LAUNCH(ctx, "delta_conv_kernel");
     // columns per lane: two when that leaves every SM a dozen warps, else one (more parallel, more instructions)
     const long long columns = (long long)d.vdim_p * d.heads * sm.n_seq;
@@ -558,14 +558,14 @@ int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const flo
 #define DSCAN(M, C)                                                                                                           \
     do {                                                                                                                      \
         constexpr int ch = M <= 4 ? 16 : 8;                                                                                   \
-        constexpr size_t smem = 2 * sizeof(float) * ch * (2 * M * 32 + 16 * C + 4);                                           \
+        constexpr size_t smem = 2 * sizeof(float) * (ch * (2 * M * 32 + 16 * C + 4) + (CH ? ch * M * 32 : 4));                \
         static bool done[16] = {};                                                                                            \
         if (!done[ctx->device & 15]) {                                                                                        \
-            CK(ctx, cudaFuncSetAttribute(delta_scan_kernel<M, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));   \
-            prefer_max_smem(delta_scan_kernel<M, C>);                                                                         \
+            CK(ctx, cudaFuncSetAttribute(delta_scan_kernel<M, C, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+            prefer_max_smem(delta_scan_kernel<M, C, CH>);                                                                     \
             done[ctx->device & 15] = true;                                                                                    \
         }                                                                                                                     \
-        CK(ctx, launch_pdl(ctx, delta_scan_kernel<M, C>, dim3((d.vdim_p + 16 * C - 1) / (16 * C), d.heads, sm.n_seq),         \
+        CK(ctx, launch_pdl(ctx, delta_scan_kernel<M, C, CH>, dim3((d.vdim_p + 16 * C - 1) / (16 * C), d.heads, sm.n_seq),     \
                            dim3(128), smem, d, proj, ldp, conv, conv_state, state, sm, heads_out));                           \
     } while (0)
 #define DSCAN_C(M)                                                                                                            \
@@ -583,14 +583,39 @@ int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const flo
 #undef DSCAN
     CK_LAUNCH(ctx, "delta_scan_kernel");
     const int units = n_rows * d.heads;
+    const float *gates = CH ? ext + d.ext() : proj + d.g_at();
+    const int ldg = CH ? 2 * d.ext() : ldp;
     if (b16) {
-        PREFER_SMEM_ONCE(delta_out_kernel<__nv_bfloat16>);
-        launch_pdl(ctx, delta_out_kernel<__nv_bfloat16>, dim3((units + 7) / 8), dim3(256), 0, d, proj, ldp, w.norm, heads_out, n_rows,
+        PREFER_SMEM_ONCE((delta_out_kernel<CH, __nv_bfloat16>));
+        launch_pdl(ctx, delta_out_kernel<CH, __nv_bfloat16>, dim3((units + 7) / 8), dim3(256), 0, d, gates, ldg, w.norm, heads_out, n_rows,
                    (__nv_bfloat16 *)out);
     } else {
-        PREFER_SMEM_ONCE(delta_out_kernel<float>);
-        launch_pdl(ctx, delta_out_kernel<float>, dim3((units + 7) / 8), dim3(256), 0, d, proj, ldp, w.norm, heads_out, n_rows, (float *)out);
+        PREFER_SMEM_ONCE((delta_out_kernel<CH, float>));
+        launch_pdl(ctx, delta_out_kernel<CH, float>, dim3((units + 7) / 8), dim3(256), 0, d, gates, ldg, w.norm, heads_out, n_rows, (float *)out);
     }
     CK_LAUNCH(ctx, "delta_out_kernel");
     return B200NN_OK;
+}
+
+}  // namespace
+
+int launch_delta_step(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const float *ext, const DeltaWeights &w, float *conv_state,
+                      float *state, const RowMap &rows, int n_rows, void *out) {
+    if (n_rows > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: more than 65535 rows");
+    if (d.dim_p > 256) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
+    if (d.channel)
+        return b16 ? step_launch<true>(ctx, d, proj, ldp, ext, w, conv_state, state, rows, n_rows, (__nv_bfloat16 *)out)
+                   : step_launch<true>(ctx, d, proj, ldp, ext, w, conv_state, state, rows, n_rows, (float *)out);
+    return b16 ? step_launch<false>(ctx, d, proj, ldp, ext, w, conv_state, state, rows, n_rows, (__nv_bfloat16 *)out)
+               : step_launch<false>(ctx, d, proj, ldp, ext, w, conv_state, state, rows, n_rows, (float *)out);
+}
+
+int launch_delta_prompt(b200nn_ctx *ctx, const DeltaDims &d, bool b16, const float *proj, int ldp, const float *ext, const DeltaWeights &w,
+                        float *conv_state, float *state, const RowMap &rows, const SeqMap &sm, int n_rows, const int *row_seq, float *conv,
+                        float *heads_out, void *out) {
+    if (d.dim_p > 256) return set_error(ctx, B200NN_ERR_UNSUPPORTED, "delta rule: dim > 256");
+    if (n_rows > 8 * 65535 || sm.n_seq > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: too many rows or sequences in a pass");
+    if (ldp & 3) return set_error(ctx, B200NN_ERR_SHAPE, "delta rule: projection rows must keep 16-byte alignment");
+    return d.channel ? prompt_launch<true>(ctx, d, b16, proj, ldp, ext, w, conv_state, state, rows, sm, n_rows, row_seq, conv, heads_out, out)
+                     : prompt_launch<false>(ctx, d, b16, proj, ldp, ext, w, conv_state, state, rows, sm, n_rows, row_seq, conv, heads_out, out);
 }

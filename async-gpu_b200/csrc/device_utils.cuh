@@ -104,6 +104,24 @@ __device__ __forceinline__ void epi_store4(const Epilogue &e, int m, int n, floa
             v = make_float4(v.x * c0.x - v.y * c0.y, v.y * c0.x + v.x * c0.y, v.z * c1.x - v.w * c1.y, v.w * c1.x + v.z * c1.y);
         }
     }
+    if (B16 && e.tail_out && n >= e.tail_at) {
+        const float f[4] = {v.x, v.y, v.z, v.w};
+        const size_t i = (size_t)m * e.tail_ld + (n - e.tail_at);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (n + j < N) {
+                if (e.tail_type == OUT_BF16) static_cast<__nv_bfloat16 *>(e.tail_out)[i + j] = __float2bfloat16_rn(f[j]);
+                else static_cast<float *>(e.tail_out)[i + j] = f[j];
+            }
+        return;
+    }
+    if (B16 && e.kv_cache && n >= e.kv_at) { // kv_w is a multiple of 16
+        if (n >= N) return;
+        const int c = n - e.kv_at, head = c / e.kv_w;
+        const size_t row = ((size_t)row_slot(e.rows, m) * e.kv_heads + head) * e.kv_cap + row_pos(e.rows, m);
+        *reinterpret_cast<uint2 *>(e.kv_cache + row * e.kv_w + (c - head * e.kv_w)) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+        return;
+    }
     const bool vec = (n + 3 < N) && ((e.ldo & 3) == 0) && (e.pos_ptr == nullptr);
     if (!vec) {
         if (n < N) epi_store<B16>(e, m, n, v.x);
@@ -349,6 +367,36 @@ __device__ __forceinline__ float load_as_float<__nv_bfloat16>(const __nv_bfloat1
 __device__ __forceinline__ void store_from_float(float *p, float v) { *p = v; }
 __device__ __forceinline__ void store_from_float(__half *p, float v) { *p = __float2half_rn(v); }
 __device__ __forceinline__ void store_from_float(__nv_bfloat16 *p, float v) { *p = __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float sigmoid_f(float v) { return 1.0f / (1.0f + expf(-v)); }
+
+// Pairs of f32 in one register pair: one instruction for two multiply-adds.
+__device__ __forceinline__ uint64_t f32x2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 f32x2_parts(uint64_t v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ void cp_async16(void *smem, const void *gmem) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+__device__ __forceinline__ void cp_async4(void *smem, const void *gmem) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
 
 // Unpacks one 32-bit word of the tiled int4 layout (nibble positions 0..7 = k offsets
 // 0,2,4,6,1,3,5,7, each stored +8) into four half2 holding the exact integers (k0,k1) (k2,k3)

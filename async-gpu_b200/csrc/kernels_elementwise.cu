@@ -558,7 +558,7 @@ int launch_tensor_transpose(b200nn_ctx *ctx, const float *in, float *out, const 
 }
 
 // ---------------------------------------------------------------------------------------------
-// Pieces of the hybrid decoder: RMS norm, embedding without positions, gated products, row gather and the
+// Pieces of the hybrid decoders: RMS norm, embedding with or without learned positions, gated products, row gather and the
 // block-diagonal f32 Linear.
 // ---------------------------------------------------------------------------------------------
 // x / sqrt(mean(x^2) + eps) * w, one block per row; output rows ldo apart.
@@ -654,20 +654,26 @@ int launch_rmsnorm(b200nn_ctx *ctx, const float *x, const float *w, float eps, i
 
 template <typename T>
 __global__ void embedding_rows_kernel(const uint32_t *__restrict__ ids, const T *__restrict__ table, int ldt, int d, int vocab,
-                                      float *__restrict__ out) {
+                                      const T *__restrict__ pos_table, int max_pos, RowMap rows, float *__restrict__ out) {
     const int r = blockIdx.x;
     pdl_trigger();
     pdl_wait();
     const uint32_t tok = min(ids[r], (uint32_t)vocab - 1); // ids are validated on the host; never read out of range
-    for (int j = threadIdx.x; j < d; j += blockDim.x) out[(size_t)r * d + j] = load_as_float<T>(table, (size_t)tok * ldt + j);
+    const size_t p = pos_table ? (size_t)min(row_pos(rows, r), max_pos - 1) * ldt : 0; // so are positions
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        const float v = load_as_float<T>(table, (size_t)tok * ldt + j);
+        out[(size_t)r * d + j] = pos_table ? v + load_as_float<T>(pos_table, p + j) : v;
+    }
 }
 int launch_embedding_rows(b200nn_ctx *ctx, const uint32_t *ids, const void *table, bool b16, int ldt, int n_rows, int d, int vocab,
-                          float *out) {
+                          const void *pos_table, int max_pos, const RowMap &rows, float *out) {
     if (n_rows <= 0) return B200NN_OK;
     PREFER_SMEM_ONCE(embedding_rows_kernel<__nv_bfloat16>);
     PREFER_SMEM_ONCE(embedding_rows_kernel<float>);
-    if (b16) launch_pdl(ctx, embedding_rows_kernel<__nv_bfloat16>, dim3(n_rows), dim3(256), 0, ids, (const __nv_bfloat16 *)table, ldt, d, vocab, out);
-    else launch_pdl(ctx, embedding_rows_kernel<float>, dim3(n_rows), dim3(256), 0, ids, (const float *)table, ldt, d, vocab, out);
+    if (b16) launch_pdl(ctx, embedding_rows_kernel<__nv_bfloat16>, dim3(n_rows), dim3(256), 0, ids, (const __nv_bfloat16 *)table, ldt, d, vocab,
+                        (const __nv_bfloat16 *)pos_table, max_pos, rows, out);
+    else launch_pdl(ctx, embedding_rows_kernel<float>, dim3(n_rows), dim3(256), 0, ids, (const float *)table, ldt, d, vocab, (const float *)pos_table, max_pos, rows,
+                    out);
     CK_LAUNCH(ctx, "embedding_rows_kernel");
     return B200NN_OK;
 }

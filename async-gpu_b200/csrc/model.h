@@ -123,6 +123,10 @@ struct LayerState {
     // delta rule: [slot][head][dim][vdim] f32 state, [slot][taps][channel] f32 convolution inputs (position
     // p in row p % taps)
     std::shared_ptr<DevBuf> state, conv;
+    // mLSTM: state as above, normaliser [slot][head][dim] and running maximum [slot][head], f32
+    std::shared_ptr<DevBuf> normaliser, maximum;
+    // differential attention: [slot][kv head][position][kv_w] keys of both maps, then the value
+    std::shared_ptr<DevBuf> kv;
 };
 
 // KV cache / state manager: `batch` sequence slots of up to `cap` positions.  Lockstep use (decode session,
@@ -161,7 +165,7 @@ struct Workspace {
     int ln_nt = 0;
     float *ln_slot(int i) const { return static_cast<float *>(ln_stats->p) + (size_t)i * rows * ln_nt * 2; }
     // hybrid models (sizes in hybrid.cu)
-    std::shared_ptr<DevBuf> proj, gate, cq, qlat, olat, heads, dstep, lin, kvx, part, meta;
+    std::shared_ptr<DevBuf> proj, gate, cq, qlat, olat, heads, dstep, lin, kvx, part, meta, low, ext, xs, y;
 };
 int workspace_alloc(b200nn_gpt2 *m, size_t rows, size_t logit_rows, Workspace *ws);
 

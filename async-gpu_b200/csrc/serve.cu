@@ -8,8 +8,9 @@
 #include "hybrid.h"
 #include "json.h"
 
-int hybrid_create(b200nn_ctx *ctx, const JsonValue &root, size_t n, const char *const *names, const float *const *data, const size_t *numels,
+int hybrid_create(b200nn_ctx *ctx, const std::string &arch, const JsonValue &root, size_t n, const char *const *names, const float *const *data, const size_t *numels,
                   uint32_t flags, b200nn_lm **out);
+bool hybrid_architecture(const std::string &arch);
 
 namespace {
 
@@ -56,11 +57,11 @@ bool to_f32(const std::string &dtype, const std::vector<char> &raw, std::vector<
 // Which builder serves an architecture name.
 enum Family { FAM_NONE, FAM_GPT2, FAM_HYBRID };
 struct { const char *name; Family family; } const REGISTRY[] = {
-    {"Vivezen", FAM_HYBRID}, {"GPT2LMHeadModel", FAM_GPT2}, {"GPT2Model", FAM_GPT2}, {"gpt2", FAM_GPT2}};
+    {"GPT2LMHeadModel", FAM_GPT2}, {"GPT2Model", FAM_GPT2}, {"gpt2", FAM_GPT2}};
 Family family_of(const std::string &arch) {
     for (const auto &e : REGISTRY)
         if (arch == e.name) return e.family;
-    return FAM_NONE;
+    return hybrid_architecture(arch) ? FAM_HYBRID : FAM_NONE;
 }
 
 }  // namespace
@@ -74,7 +75,7 @@ extern "C" int32_t b200nn_lm_create(b200nn_ctx *ctx, const char *config_json, si
     const std::string arch = architecture_of(root);
     if (family_of(arch) != FAM_HYBRID)
         return set_error(ctx, B200NN_ERR_UNSUPPORTED, "no model family builds architecture '" + arch + "' from host tensors");
-    return hybrid_create(ctx, root, n_tensors, names, data, numels, flags, out);
+    return hybrid_create(ctx, arch, root, n_tensors, names, data, numels, flags, out);
 }
 
 extern "C" int32_t b200nn_lm_load(b200nn_ctx *ctx, const char *dir, uint32_t flags, b200nn_lm **out) {
@@ -118,7 +119,7 @@ extern "C" int32_t b200nn_lm_load(b200nn_ctx *ctx, const char *dir, uint32_t fla
         data.push_back(store[i].data());
         numels.push_back(store[i].size());
     }
-    return hybrid_create(ctx, root, names.size(), names.data(), data.data(), numels.data(), flags, out);
+    return hybrid_create(ctx, arch, root, names.size(), names.data(), data.data(), numels.data(), flags, out);
 }
 
 extern "C" b200nn_lm *b200nn_gpt2_as_lm(b200nn_gpt2 *m) { return m; }
