@@ -79,6 +79,19 @@ class _DeltaWeights(C.Structure):
     _fields_ = [(n, C.c_void_p) for n in ("conv", "a_exp", "dt_bias", "norm")]
 
 
+class _MlstmShape(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("heads", "dim", "vdim")] + [(n, C.c_float) for n in ("gate_cap", "eps")]
+
+
+class _MlstmWeights(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("i_bias", "f_bias", "norm")]
+
+
+class _DiffShape(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "temp_every")] + [
+        (n, C.c_float) for n in ("scale", "softcap", "temp_coef", "lam", "diff", "eps")]
+
+
 class _Weights(C.Structure):
     _fields_ = [("wte", _f32p), ("wpe", _f32p), ("ln_f_weight", _f32p), ("ln_f_bias", _f32p),
                 ("layers", C.POINTER(_LayerW))]
@@ -209,6 +222,11 @@ def load_library() -> C.CDLL:
             "b200nn_latent_decode_attention": (i32, [vp, C.POINTER(_LatentShape), u32, vp, vp, vp, i32, vp, vp, i32, i32, i32, vp]),
             "b200nn_delta_rule": (i32, [vp, C.POINTER(_DeltaShape), u32, vp, C.POINTER(_DeltaWeights), vp, vp, vp, vp, i32, i32, i32,
                                         vp, vp, vp]),
+            "b200nn_channel_delta_rule": (i32, [vp, C.POINTER(_DeltaShape), u32, vp, vp, C.POINTER(_DeltaWeights), vp, vp, vp, vp, i32, i32,
+                                                i32, vp, vp, vp]),
+            "b200nn_mlstm": (i32, [vp, C.POINTER(_MlstmShape), u32, vp, C.POINTER(_MlstmWeights), vp, vp, vp, vp, vp, i32, i32, vp, vp, vp]),
+            "b200nn_diff_attention": (i32, [vp, C.POINTER(_DiffShape), u32, vp, vp, i32, i32, vp, vp, vp, i32, i32, i32, vp, vp]),
+            "b200nn_stream_step": (i32, [vp, u32, i32, i32, i32, vp, vp, vp, vp, vp, vp, C.c_float, vp, vp]),
             "b200nn_bpe_load": (i32, [C.c_char_p, u32, vpp]),
             "b200nn_bpe_create": (i32, [C.c_char_p, szp, _u32p, sz, u32, vpp]),
             "b200nn_bpe_destroy": (None, [vp]), "b200nn_bpe_vocab_size": (sz, [vp]),

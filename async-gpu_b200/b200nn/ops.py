@@ -6,7 +6,8 @@ import ctypes as C
 import numpy as np
 
 from . import (ACT_GELU_SIGMOID, ACT_GELU_TANH, ACT_RELU, ACT_SIGMOID, ACT_SILU, ERR_SHAPE, GpuTensor, KernelRegistry, NnError, _f32,
-               _f32p, _out, _u32p, _DeltaShape, _DeltaWeights, _LatentShape, load_library)
+               _f32p, _out, _u32p, _DeltaShape, _DeltaWeights, _DiffShape, _LatentShape,
+               _MlstmShape, _MlstmWeights, load_library)
 
 
 # ---- quantize (ops/quantize.rs) ----
@@ -224,3 +225,32 @@ def delta_rule(shape, weights, proj_ptr, conv_state_ptr, state_ptr, pos_ptr, slo
     (conv, a_exp, dt_bias, norm).  ``n_seq`` 0: one token per row, else prompt portions."""
     reg.check(reg.lib.b200nn_delta_rule(reg.h, C.byref(_DeltaShape(*shape)), flags, proj_ptr, C.byref(_DeltaWeights(*weights)), conv_state_ptr,
                                         state_ptr, pos_ptr, slot_ptr, n_rows, n_seq, max_n, seq_ptr, scratch_ptr, out_ptr))
+
+
+def channel_delta_rule(shape, weights, proj_ptr, ext_ptr, conv_state_ptr, state_ptr, pos_ptr, slot_ptr, n_rows, out_ptr, reg, n_seq=0, max_n=0,
+                       seq_ptr=None, scratch_ptr=None, flags=0):
+    """The same with a decay per key channel and a sigmoid gate, whose inputs are ``ext``; dt_bias is [heads][dim]."""
+    reg.check(reg.lib.b200nn_channel_delta_rule(reg.h, C.byref(_DeltaShape(*shape)), flags, proj_ptr, ext_ptr, C.byref(_DeltaWeights(*weights)),
+                                                conv_state_ptr, state_ptr, pos_ptr, slot_ptr, n_rows, n_seq, max_n, seq_ptr, scratch_ptr, out_ptr))
+
+
+def mlstm(shape, weights, proj_ptr, memory_ptr, normaliser_ptr, maximum_ptr, pos_ptr, slot_ptr, n_rows, out_ptr, reg, n_seq=0, seq_ptr=None,
+          scratch_ptr=None, flags=0):
+    """Matrix memory with exponential gates; ``shape`` is (heads, dim, vdim, gate_cap, eps), ``weights`` the device
+    pointers (i_bias, f_bias, norm).  ``n_seq`` 0: one token per row, else prompt portions."""
+    reg.check(reg.lib.b200nn_mlstm(reg.h, C.byref(_MlstmShape(*shape)), flags, proj_ptr, C.byref(_MlstmWeights(*weights)), memory_ptr, normaliser_ptr,
+                                   maximum_ptr, pos_ptr, slot_ptr, n_rows, n_seq, seq_ptr, scratch_ptr, out_ptr))
+
+
+def diff_attention(shape, q_ptr, cache_ptr, capacity, n_slots, pos_ptr, slot_ptr, gate_ptr, n_rows, out_ptr, reg, n_seq=0, max_n=0, seq_ptr=None,
+                   flags=0):
+    """Differential attention against cached keys and values; ``shape`` is (heads, kv_heads, dim, vdim, temp_every, scale,
+    softcap, temp_coef, lam, diff, eps).  ``n_seq`` 0: one row per sequence, else prompt portions."""
+    reg.check(reg.lib.b200nn_diff_attention(reg.h, C.byref(_DiffShape(*shape)), flags, q_ptr, cache_ptr, capacity, n_slots, pos_ptr, slot_ptr, gate_ptr,
+                                            n_rows, n_seq, max_n, seq_ptr, out_ptr))
+
+
+def stream_step(n_rows, streams, width, xs_ptr, x0_ptr, y_ptr, prev_ptr, next_ptr, norm_ptr, eps, out_ptr, sum_out_ptr, reg, flags=0):
+    """Update of the residual streams, then the next sublayer's normalised input (or the sum of the streams)."""
+    reg.check(reg.lib.b200nn_stream_step(reg.h, flags, n_rows, streams, width, xs_ptr, x0_ptr, y_ptr, prev_ptr, next_ptr, norm_ptr, eps, out_ptr,
+                                         sum_out_ptr))

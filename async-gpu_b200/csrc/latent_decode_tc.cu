@@ -26,7 +26,7 @@
 
 #include "device_utils.cuh"
 #include "hybrid.h"
-#include "tc_ptx.cuh"
+#include "tc_decode.cuh"
 
 namespace {
 
@@ -40,54 +40,6 @@ struct Bars {
     uint64_t q_full, r_full, r_empty, s_full, p_full, o_full;
     uint64_t c_full[MAX_PAIRS], c_empty[MAX_PAIRS];
 };
-
-// Butterfly over the warp that also transposes: on return v[0] of lane l holds the reduction over all lanes of
-// column l (N = 32) or l >> 1 (N = 16).
-template <int N, bool MAX>
-__device__ __forceinline__ void reduce_columns(float (&v)[N]) {
-    const int lane = threadIdx.x & 31;
-    int o = 16;
-#pragma unroll
-    for (int w = N / 2; w >= 1; w >>= 1, o >>= 1) {
-        const bool up = (lane & o) != 0;
-#pragma unroll
-        for (int i = 0; i < w; ++i) {
-            const float send = up ? v[i] : v[i + w], keep = up ? v[i + w] : v[i];
-            const float r = __shfl_xor_sync(0xffffffffu, send, o);
-            v[i] = MAX ? fmaxf(keep, r) : keep + r;
-        }
-    }
-    if (N == 16) {
-        const float r = __shfl_xor_sync(0xffffffffu, v[0], 1);
-        v[0] = MAX ? fmaxf(v[0], r) : v[0] + r;
-    }
-}
-
-__device__ __forceinline__ void bar_softmax() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
-// The same with a vote: every thread learns whether any of them wants to give up.
-__device__ __forceinline__ bool bar_softmax_any(bool pred) {
-    uint32_t r;
-    asm volatile(
-        "{\n\t.reg .pred p, q;\n\t"
-        "setp.ne.u32 q, %1, 0;\n\t"
-        "bar.red.or.pred p, 1, 128, q;\n\t"
-        "selp.u32 %0, 1, 0, p;\n\t}"
-        : "=r"(r)
-        : "r"((uint32_t)pred)
-        : "memory");
-    return r != 0;
-}
-
-template <int N>
-__device__ __forceinline__ void tmem_ld_cols(uint32_t addr, float (&f)[N]) {
-#pragma unroll
-    for (int c = 0; c < N; c += 16) {
-        uint32_t v[16];
-        tc::tmem_ld_x16(addr + c, v);
-#pragma unroll
-        for (int i = 0; i < 16; ++i) f[c + i] = __uint_as_float(v[i]);
-    }
-}
 
 struct DecodeTcArgs {
     LatentDims d;
@@ -257,19 +209,19 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_c, const __grid_c
         bool ok = true;
         for (int j = 0; j < n_tiles; ++j) {
             ok = tc::mbar_wait(bar(bars.s_full), j & 1, &abort_flag, a.dev_err, ERR_LD_S);
-            ok = !bar_softmax_any(!ok); // all four warps go on or none does; red is free again
+            ok = !tc::bar_softmax_any(!ok); // all four warps go on or none does; red is free again
             if (!ok) break;
             tc::tc_fence_after_sync();
             float v[N], t[N];
-            tmem_ld_cols<N>(lane_base, v);
+            tc::tmem_ld_cols<N>(lane_base, v);
             const int kp = (t0 + j) * 128 + key;
             const bool vis = kp >= first && kp <= pos;
 #pragma unroll
             for (int h = 0; h < N; ++h) t[h] = v[h] = vis ? v[h] * a.scale_log2e : -INFINITY;
-            reduce_columns<N, true>(t);
+            tc::reduce_columns<N, true>(t);
             if (N == 32) red[quad][lane] = t[0];
             else if (!(lane & 1)) red[quad][lane >> 1] = t[0];
-            bar_softmax();
+            tc::bar_softmax();
             bool moved = false;
 #pragma unroll
             for (int h = 0; h < N; ++h) {
@@ -305,13 +257,13 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_c, const __grid_c
             tc::tc_fence_before_sync();
             tc::mbar_arrive(bar(bars.p_full));
         }
-        bar_softmax();
+        tc::bar_softmax();
         if (ok) { // sums over the keys
-            reduce_columns<N, false>(l);
+            tc::reduce_columns<N, false>(l);
             if (N == 32) red[quad][lane] = l[0];
             else if (!(lane & 1)) red[quad][lane >> 1] = l[0];
         }
-        bar_softmax();
+        tc::bar_softmax();
         if (ok && n_tiles > 0) {
             ok = tc::mbar_wait(bar(bars.o_full), 0, &abort_flag, a.dev_err, ERR_LD_O);
             tc::tc_fence_after_sync();
@@ -329,7 +281,7 @@ latent_decode_tc_kernel(const __grid_constant__ CUtensorMap tm_c, const __grid_c
             }
             if (n_tiles > 0)
                 for (int i = 0; i < tp; ++i) {
-                    tmem_ld_cols<N>(lane_base + N * (1 + i), m); // the maxima are not needed any more
+                    tc::tmem_ld_cols<N>(lane_base + N * (1 + i), m); // the maxima are not needed any more
                     const int c = i * 128 + key;
                     if (c < d.rank_p)
 #pragma unroll

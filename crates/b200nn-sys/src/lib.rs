@@ -133,6 +133,43 @@ pub struct b200nn_delta_weights {
     pub norm: *const f32,
 }
 
+/// Sizes and constants of the matrix memory with exponential gates (mLSTM).
+#[repr(C)]
+#[derive(Clone, Copy, Debug, PartialEq)]
+pub struct b200nn_mlstm_shape {
+    pub heads: i32,
+    pub dim: i32,
+    pub vdim: i32,
+    pub gate_cap: f32,
+    pub eps: f32,
+}
+
+/// Device pointers of the mLSTM's small weights.
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct b200nn_mlstm_weights {
+    pub i_bias: *const f32,
+    pub f_bias: *const f32,
+    pub norm: *const f32,
+}
+
+/// Sizes and constants of differential attention.
+#[repr(C)]
+#[derive(Clone, Copy, Debug, PartialEq)]
+pub struct b200nn_diff_shape {
+    pub heads: i32,
+    pub kv_heads: i32,
+    pub dim: i32,
+    pub vdim: i32,
+    pub temp_every: i32,
+    pub scale: f32,
+    pub softcap: f32,
+    pub temp_coef: f32,
+    pub lam: f32,
+    pub diff: f32,
+    pub eps: f32,
+}
+
 /// `TransformerLayerWeights` (model.rs:112-139): host f32, dense weights in Conv1D layout [in,out].
 #[repr(C)]
 #[derive(Clone, Copy)]
@@ -823,6 +860,74 @@ extern "C" {
         seq_dev: *const i32,
         scratch_dev: *mut f32,
         out_dev: *mut c_void,
+    ) -> i32;
+    pub fn b200nn_channel_delta_rule(
+        ctx: *mut b200nn_ctx,
+        shape: *const b200nn_delta_shape,
+        flags: u32,
+        proj_dev: *const f32,
+        ext_dev: *const f32,
+        w: *const b200nn_delta_weights,
+        conv_state_dev: *mut f32,
+        state_dev: *mut f32,
+        pos_dev: *const i32,
+        slot_dev: *const i32,
+        n_rows: i32,
+        n_seq: i32,
+        max_n: i32,
+        seq_dev: *const i32,
+        scratch_dev: *mut f32,
+        out_dev: *mut c_void,
+    ) -> i32;
+    pub fn b200nn_mlstm(
+        ctx: *mut b200nn_ctx,
+        shape: *const b200nn_mlstm_shape,
+        flags: u32,
+        proj_dev: *const f32,
+        w: *const b200nn_mlstm_weights,
+        memory_dev: *mut f32,
+        normaliser_dev: *mut f32,
+        maximum_dev: *mut f32,
+        pos_dev: *const i32,
+        slot_dev: *const i32,
+        n_rows: i32,
+        n_seq: i32,
+        seq_dev: *const i32,
+        scratch_dev: *mut f32,
+        out_dev: *mut c_void,
+    ) -> i32;
+    pub fn b200nn_diff_attention(
+        ctx: *mut b200nn_ctx,
+        shape: *const b200nn_diff_shape,
+        flags: u32,
+        q_dev: *const c_void,
+        cache_dev: *const c_void,
+        capacity: i32,
+        n_slots: i32,
+        pos_dev: *const i32,
+        slot_dev: *const i32,
+        gate_dev: *const f32,
+        n_rows: i32,
+        n_seq: i32,
+        max_n: i32,
+        seq_dev: *const i32,
+        out_dev: *mut c_void,
+    ) -> i32;
+    pub fn b200nn_stream_step(
+        ctx: *mut b200nn_ctx,
+        flags: u32,
+        n_rows: i32,
+        streams: i32,
+        width: i32,
+        xs_dev: *mut f32,
+        x0_dev: *const f32,
+        y_dev: *const f32,
+        prev_dev: *const f32,
+        next_dev: *const f32,
+        norm_dev: *const f32,
+        eps: f32,
+        out_dev: *mut c_void,
+        sum_out_dev: *mut f32,
     ) -> i32;
     pub fn b200nn_bpe_load(path: *const c_char, endoftext_id: u32, out: *mut *mut b200nn_bpe) -> i32;
     pub fn b200nn_bpe_create(

@@ -517,11 +517,11 @@ B200NN_API int32_t b200nn_gpt2_load_safetensors(b200nn_ctx *ctx, const char *pat
 
 /* ---- language models by architecture: registry, cache slots, serving step --------------------------
  * b200nn_lm is a decoder-only model of any family: GPT-2 (a view of a b200nn_gpt2), or a hybrid decoder
- * whose layers (gated delta rule or latent attention, each with an optional gated feed-forward) are listed in
- * a config.json.  No counterpart in the reference, whose models are separate Rust types.
+ * whose layers (gated delta rule, mLSTM, latent or differential attention, each with an optional gated feed-forward) are
+ * listed in a config.json.  No counterpart in the reference, whose models are separate Rust types.
  *   _create  config_json (the text) plus host f32 tensors by name
  *   _load    a folder with config.json and model.safetensors (F32, F16 or BF16); the family follows from
- *            the configuration's "architecture" ("Vivezen"), or its "architectures" / "model_type" (GPT-2)
+ *            the configuration's "architecture" ("Vivezen", "Zufilorn"), or its "architectures" / "model_type" (GPT-2)
  * Default precision of hybrid models: bfloat16 weights and activations, f32 accumulation, norms, softmax,
  * recurrence and residual; B200NN_LM_F32 selects f32 throughout (GPT-2 refuses it: B200NN_ERR_UNSUPPORTED). */
 typedef struct {
@@ -594,6 +594,51 @@ B200NN_API int32_t b200nn_delta_rule(b200nn_ctx *ctx, const b200nn_delta_shape *
                                      const b200nn_delta_weights *w, float *conv_state_dev, float *state_dev, const int32_t *pos_dev,
                                      const int32_t *slot_dev, int32_t n_rows, int32_t n_seq, int32_t max_n, const int32_t *seq_dev,
                                      float *scratch_dev, void *out_dev);
+/* The same rule with one decay per head and key channel and a sigmoid output gate.  proj f32 [n_rows] x ([kv_heads][dim] q,
+ * [kv_heads][dim] k, [heads][vdim] v, [heads] step-size inputs, then padding to a multiple of 16); ext f32 [n_rows] x (decay
+ * inputs [heads][dim], gate inputs [heads][vdim], each part padded to heads * max(dim, vdim) columns); dt_bias
+ * [heads][dim].  The rest as above; scratch f32 of n_rows * (2 kv_heads dim + 2 heads vdim + heads dim + heads + kv_heads + 4). */
+B200NN_API int32_t b200nn_channel_delta_rule(b200nn_ctx *ctx, const b200nn_delta_shape *shape, uint32_t flags, const float *proj_dev,
+                                             const float *ext_dev, const b200nn_delta_weights *w, float *conv_state_dev,
+                                             float *state_dev, const int32_t *pos_dev, const int32_t *slot_dev, int32_t n_rows,
+                                             int32_t n_seq, int32_t max_n, const int32_t *seq_dev, float *scratch_dev, void *out_dev);
+/* Matrix memory with exponential gates (mLSTM), its output norm and gate.  proj f32 [n_rows] x ([heads][dim] q, [heads][dim] k,
+ * [heads][vdim] v, [heads][vdim] gate, [heads] input gates, [heads] forget gates, then padding to a multiple of 4);
+ * weights f32 on the device: i_bias, f_bias [heads], norm [heads][vdim]; memory f32 [slots][heads][dim][vdim], normaliser
+ * [slots][heads][dim], maximum [slots][heads]; out [n_rows][heads][vdim].  n_seq 0: one token per row.  Else prompt
+ * portions: seq [4][n_seq] (slot, first row, rows, past) and scratch f32 of n_rows * heads * (vdim + 4). */
+typedef struct {
+    int32_t heads, dim, vdim;
+    float gate_cap, eps;
+} b200nn_mlstm_shape;
+typedef struct {
+    const float *i_bias, *f_bias, *norm;
+} b200nn_mlstm_weights;
+B200NN_API int32_t b200nn_mlstm(b200nn_ctx *ctx, const b200nn_mlstm_shape *shape, uint32_t flags, const float *proj_dev,
+                                const b200nn_mlstm_weights *w, float *memory_dev, float *normaliser_dev, float *maximum_dev,
+                                const int32_t *pos_dev, const int32_t *slot_dev, int32_t n_rows, int32_t n_seq, const int32_t *seq_dev,
+                                float *scratch_dev, void *out_dev);
+/* Differential attention: two softmax maps per head over the same values, (a1 - lam a2) over its root mean square times
+ * (1 - diff) times sigmoid(gate).  q [n_rows][heads][2][dim]; cache [n_slots][kv_heads][capacity] rows of 2 dim key and
+ * vdim value columns, the rows' own positions already in it; gate f32 [n_rows][heads]; pos and slot per row (slot NULL: slot = row); out
+ * [n_rows][heads][vdim].  Scores are (q . k) * scale * (1 + temp_coef ln(floor((pos + 1) / temp_every) + 1)), then softcap
+ * tanh(score / softcap) (softcap 0: none).  n_seq 0: one row per sequence.  Else seq [4][n_seq]: slot, first row, rows
+ * (the largest is max_n), past. */
+typedef struct {
+    int32_t heads, kv_heads, dim, vdim, temp_every;
+    float scale, softcap, temp_coef, lam, diff, eps;
+} b200nn_diff_shape;
+B200NN_API int32_t b200nn_diff_attention(b200nn_ctx *ctx, const b200nn_diff_shape *shape, uint32_t flags, const void *q_dev,
+                                         const void *cache_dev, int32_t capacity, int32_t n_slots, const int32_t *pos_dev,
+                                         const int32_t *slot_dev, const float *gate_dev, int32_t n_rows, int32_t n_seq, int32_t max_n,
+                                         const int32_t *seq_dev, void *out_dev);
+/* Residual streams between two sublayers.  xs f32 [n_rows][streams][width], updated in place: with y (f32 [n_rows][width])
+ * x_t <- sum_s mix[s][t] x_s + out[t] y, without it x_t <- x0.  Then out = RMS norm (times norm [width]) of sum_s in[s] x_s;
+ * or, with sum_out (f32 [n_rows][width]), only the sum of the streams is written there.  prev and next: f32 [streams]
+ * in, [streams] out, [streams from][streams to] mix of the sublayer before and after. */
+B200NN_API int32_t b200nn_stream_step(b200nn_ctx *ctx, uint32_t flags, int32_t n_rows, int32_t streams, int32_t width, float *xs_dev,
+                                      const float *x0_dev, const float *y_dev, const float *prev_dev, const float *next_dev,
+                                      const float *norm_dev, float eps, void *out_dev, float *sum_out_dev);
 
 /* ---- Gpt2Tokenizer (crates/core/gpu-host/src/tokenizer.rs:34-62) ---------------------------------
  * Host code.  The reference wraps tiktoken-rs' r50k_base; here the byte-level BPE is implemented over a

@@ -50,7 +50,7 @@ def test_rust_sys_crate_declares_exactly_the_header():
     # struct fields: C `const float *a, *b;` lists against Rust `pub a: *const f32,`
     for name in ("b200nn_gpt2_config", "b200nn_gpt2_layer_weights", "b200nn_gpt2_weights", "b200nn_block_weights",
                  "b200nn_gpt2_diagnostic", "b200nn_lm_info", "b200nn_latent_shape",
-                 "b200nn_delta_shape", "b200nn_delta_weights"):
+                 "b200nn_delta_shape", "b200nn_delta_weights", "b200nn_mlstm_shape", "b200nn_mlstm_weights", "b200nn_diff_shape"):
         c_body = re.search(r"typedef struct \{([^}]*)\}\s*" + name + r"\s*;", header).group(1)
         c_fields = []
         for stmt in c_body.split(";"):
