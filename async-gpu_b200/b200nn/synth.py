@@ -145,3 +145,71 @@ def hybrid_weights(cfg, base_seed=BASE_SEED):
             mat(p + "mlp.up", ff, d)
             mat(p + "mlp.down", d, ff)
     return out
+
+
+def zufilorn_config(width, layers, vocab, heads, kv_heads, dim, vdim, ff, positions, streams=2, conv=4):
+    """config.json of a Zufilorn decoder whose layers repeat channel delta rule, mLSTM, mLSTM, differential attention, all
+    with a feed-forward (mixer heads of vdim x vdim states; attention maps of dim columns over vdim values)."""
+    mlp = {"kind": "dense", "ff": ff}
+    dlt = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": vdim, "vdim": vdim, "conv": conv}}
+    mem = {"type": "mlstm", "mlp": mlp, "mixer": {"heads": heads, "dim": vdim, "vdim": vdim, "gate_cap": 15.0}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5,
+                                                      "softcap": 30.0, "q_temp": {"coef": 0.1, "every": 1024}, "diff": 0.5}}
+    return {"architecture": "Zufilorn", "width": width, "vocab": vocab, "streams": streams, "max_positions": positions, "norm": {"eps": 1e-5},
+            "layers": [(dlt, mem, mem, att)[i % 4] for i in range(layers)]}
+
+
+def zufilorn_weights(cfg, rank, base_seed=BASE_SEED):
+    """Random f32 weights of a Zufilorn decoder by tensor name: matrices with unit row gain, norms of one, decays and gates
+    spread from a few tokens to hundreds; rank: inner size of the two-step projections."""
+    d, n, out = cfg["width"], cfg["streams"], {}
+
+    def mat(name, *shape):
+        out[name] = np.random.default_rng(base_seed + len(out)).standard_normal(shape, dtype=np.float32) * np.float32(shape[-1] ** -0.5)
+
+    def full(name, value, *shape):
+        out[name] = np.full(shape, value, dtype=np.float32)
+
+    mat("embed", cfg["vocab"], d)
+    mat("head", cfg["vocab"], d)
+    mat("pos", cfg["max_positions"], d)
+    full("final.norm", 0.0, d)
+    for i, layer in enumerate(cfg["layers"]):
+        p, x = f"l{i}.", layer["mixer"]
+        m, H, dim, vd = p + "mix.", x["heads"], x["dim"], x["vdim"]
+        full(p + "norm1", 0.0, d)
+        if layer["type"] == "channel_delta":
+            KH = x["kv_heads"]
+            for t, c in (("q", KH * dim), ("k", KH * dim), ("v", H * vd)):
+                mat(m + t, c, d)
+                mat(m + t + ".conv", c, x["conv"])
+            for t, r, c in (("b", H, d), ("a1", rank, d), ("a2", H * dim, rank), ("g1", rank, d), ("g2", H * vd, rank)):
+                mat(m + t, r, c)
+            out[m + "A_log"] = np.linspace(-4.0, 0.5, H, dtype=np.float32)
+            full(m + "dt_bias", -1.0, H * dim)
+            full(m + "norm", 1.0, vd)
+        elif layer["type"] == "mlstm":
+            for t, c in (("q", H * dim), ("k", H * dim), ("v", H * vd), ("g", H * vd), ("i", H), ("f", H)):
+                mat(m + t, c, d)
+            full(m + "i.b", 0.0, H)
+            out[m + "f.b"] = np.linspace(2.0, 6.0, H, dtype=np.float32)
+            full(m + "norm", 1.0, H * vd)
+        else:
+            G = x["kv_heads"]
+            for t, c in (("q", H * 2 * dim), ("k", G * 2 * dim), ("v", G * vd), ("g", H)):
+                mat(m + t, c, d)
+            for t in ("lq1", "lk1", "lq2", "lk2"):
+                mat(m + t, dim)
+        mat(m + "o", d, H * vd)
+        sub = 1
+        if layer.get("mlp"):
+            ff, sub = layer["mlp"]["ff"], 2
+            full(p + "norm2", 0.0, d)
+            mat(p + "mlp.gate", ff, d)
+            mat(p + "mlp.up", ff, d)
+            mat(p + "mlp.down", d, ff)
+        for q in range(1, sub + 1):
+            full(f"{p}hc{q}.in", 1.0 / n, n)
+            full(f"{p}hc{q}.out", 1.0, n)
+            out[f"{p}hc{q}.mix"] = np.eye(n, dtype=np.float32)
+    return out

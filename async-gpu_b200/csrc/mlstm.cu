@@ -20,6 +20,9 @@ namespace {
 __device__ __forceinline__ float soft_cap(float v, float cap) { return cap * tanhf(v / cap); }
 __device__ __forceinline__ float log_sigmoid_f(float v) { return fminf(v, 0.0f) - log1pf(expf(-fabsf(v))); }
 
+// output gate (not part of the recurrence): fast exponential and division
+__device__ __forceinline__ float gate_f(float v) { return __fdividef(1.0f, 1.0f + __expf(-v)); }
+
 // ---- decoding ----------------------------------------------------------------------------------------
 // Block = (row, head), eight warps; warp w holds state rows w, w + 8, ..., lane l columns 4l .. 4l+3 of a 128-column
 // chunk.  Under the state's loads the threads fetch q, k, v, the gates and their entry of the normaliser.
@@ -112,32 +115,31 @@ mlstm_step_kernel(MlstmDims d, const float *__restrict__ proj, int ldp, MlstmWei
     const float rn = inv / sqrtf(warp_sum(s) / (float)d.vdim + d.eps);
     for (int j = lane; j < d.vdim; j += 32)
         store_from_float(out + ((size_t)row * d.heads + h) * d.vdim_p + j,
-                         so[j] * rn * w.norm[h * d.vdim_p + j] * sigmoid_f(p[d.g_at() + h * d.vdim_p + j]));
+                         so[j] * rn * w.norm[h * d.vdim_p + j] * gate_f(p[d.g_at() + h * d.vdim_p + j]));
 }
 
 // ---- prompts -----------------------------------------------------------------------------------------
-// One warp per (head, sequence).  A token maps m to max(f + m, i); maps compose as (f1 + f2, max(i1 + f2, i2)), so 32
-// tokens are one warp scan.  gates [row][head]: keep e^(f + m - m'), write e^(i - m'), floor e^(-m'), and room for n . q.
-__global__ void __launch_bounds__(32)
+// Block = (head, sequence), eight warps, each with a contiguous segment of the tokens.  A token maps m to max(f + m, i); maps
+// compose as (f1 + f2, max(i1 + f2, i2)), so 32 tokens are one warp scan and a segment is one map: the first pass over the
+// tokens makes the segments' maps, the second starts from the maximum that enters its segment.  gates [row][head]: keep
+// e^(f + m - m'), write e^(i - m'), floor e^(-m'), and room for n . q.
+__global__ void __launch_bounds__(256)
 mlstm_gate_kernel(MlstmDims d, const float *__restrict__ proj, int ldp, MlstmWeights w, MlstmState state, SeqMap sm, float4 *__restrict__ gates) {
-    const int h = blockIdx.x, sidx = blockIdx.y, lane = threadIdx.x;
+    __shared__ float2 seg[8];
+    const int h = blockIdx.x, sidx = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     pdl_trigger();
     const float ib = w.i_bias[h], fb = w.f_bias[h];
     pdl_wait();
-    const int n = sm.n[sidx], row0 = sm.row0[sidx];
+    const int n = sm.n[sidx], row0 = sm.row0[sidx], per = (n + 255) / 256 * 32, t_beg = warp * per, t_end = min(n, t_beg + per);
     float *mp = state.maximum + (size_t)sm.slot[sidx] * d.heads + h;
     float m = sm.past[sidx] > 0 ? *mp : 0.0f;
-    auto fetch = [&](int t, float &i, float &f) {
+    float i = 0.0f, f = 0.0f, a, b;
+    auto scan = [&](int t) { // the lane's gates and the map from the group's start through its token; past the end the map is the identity
         const float *p = proj + (size_t)(row0 + min(t, n - 1)) * ldp;
-        i = p[d.i_at() + h];
-        f = p[d.f_at() + h];
-    };
-    float i_next, f_next;
-    fetch(lane, i_next, f_next);
-    for (int t0 = 0; t0 < n; t0 += 32) {
-        const float i = soft_cap(i_next + ib, d.cap), f = log_sigmoid_f(soft_cap(f_next + fb, d.cap));
-        fetch(t0 + 32 + lane, i_next, f_next);
-        float a = f, b = i;
+        i = soft_cap(p[d.i_at() + h] + ib, d.cap);
+        f = log_sigmoid_f(soft_cap(p[d.f_at() + h] + fb, d.cap));
+        a = t < t_end ? f : 0.0f;
+        b = t < t_end ? i : -INFINITY;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float pa = __shfl_up_sync(0xffffffffu, a, o), pb = __shfl_up_sync(0xffffffffu, b, o);
@@ -146,15 +148,28 @@ mlstm_gate_kernel(MlstmDims d, const float *__restrict__ proj, int ldp, MlstmWei
                 a += pa;
             }
         }
+    };
+    float sa = 0.0f, sb = -INFINITY;
+    for (int t0 = t_beg; t0 < t_end; t0 += 32) {
+        scan(t0 + lane);
+        const float ga = __shfl_sync(0xffffffffu, a, 31), gb = __shfl_sync(0xffffffffu, b, 31);
+        sb = fmaxf(sb + ga, gb);
+        sa += ga;
+    }
+    if (lane == 0) seg[warp] = make_float2(sa, sb);
+    __syncthreads(); // every warp has also read the maximum the sequence came with
+    for (int s = 0; s < warp; ++s) m = fmaxf(seg[s].x + m, seg[s].y);
+    for (int t0 = t_beg; t0 < t_end; t0 += 32) {
+        scan(t0 + lane);
         const float m_new = fmaxf(a + m, b);
         float m_old = __shfl_up_sync(0xffffffffu, m_new, 1);
         if (lane == 0) m_old = m;
         // from the maxima as they were rounded, so that their errors cancel along the sequence
-        if (t0 + lane < n)
+        if (t0 + lane < t_end)
             gates[(size_t)(row0 + t0 + lane) * d.heads + h] = make_float4(expf(f + m_old - m_new), expf(i - m_new), expf(-m_new), 0.0f);
-        m = __shfl_sync(0xffffffffu, m_new, min(31, n - 1 - t0));
+        m = __shfl_sync(0xffffffffu, m_new, 31);
     }
-    if (lane == 0) *mp = m;
+    if (lane == 0 && t_end == n && t_beg < n) *mp = m;
 }
 
 // Block = (16 NC state columns, head, sequence), four warps; the eight lanes of a column group hold its dim entries
@@ -197,16 +212,16 @@ mlstm_scan_kernel(MlstmDims d, const float *__restrict__ proj, int ldp, MlstmSta
             }
         }
     auto copy = [&](int t0, Stage &st) {
-        const int nt = min(TOK, n - t0), dv = d.dim_p >> 2, cv = norm ? 0 : min(CB, d.vdim_p - cg * CB) >> 2;
-        const float *c = proj + (size_t)(row0 + t0) * ldp;
-        for (int i = tid; i < nt * dv; i += 128) {
-            const int t = i / dv, j = (i - t * dv) * 4;
-            cp_async16(&st.q[t][j], c + (size_t)t * ldp + d.q_at() + h * d.dim_p + j);
-            cp_async16(&st.k[t][j], c + (size_t)t * ldp + d.k_at() + h * d.dim_p + j);
-        }
-        for (int i = tid; i < nt * cv; i += 128) {
-            const int t = i / cv, j = (i - t * cv) * 4;
-            cp_async16(&st.v[t][j], c + (size_t)t * ldp + d.v_at() + h * d.vdim_p + cg * CB + j);
+        const int nt = min(TOK, n - t0), cv = norm ? 0 : min(CB, d.vdim_p - cg * CB);
+        for (int t = warp; t < nt; t += 4) { // a warp per token
+            const float *c = proj + (size_t)(row0 + t0 + t) * ldp;
+#pragma unroll
+            for (int j = lane * 4; j < DP; j += 128)
+                if (j < d.dim_p) {
+                    cp_async16(&st.q[t][j], c + d.q_at() + h * d.dim_p + j);
+                    cp_async16(&st.k[t][j], c + d.k_at() + h * d.dim_p + j);
+                }
+            if (lane * 4 < cv) cp_async16(&st.v[t][lane * 4], c + d.v_at() + h * d.vdim_p + cg * CB + lane * 4);
         }
         if (tid < nt) { // keep and write only: the other half of the row is being written by the normaliser's block
             const float *g = reinterpret_cast<const float *>(gates + (size_t)(row0 + t0 + tid) * d.heads + h);
@@ -232,51 +247,63 @@ mlstm_scan_kernel(MlstmDims d, const float *__restrict__ proj, int ldp, MlstmSta
         __syncthreads();
         const Stage &st = stages[b];
         const int nt = norm && warp ? 0 : min(TOK, n - t0);
-#pragma unroll 4
-        for (int t = 0; t < nt; ++t) {
-            const float2 sc = *reinterpret_cast<const float2 *>(st.s[t]);
-            G *= sc.x;
-            if (G < 9.5367431640625e-7f) { // the same in every thread of the block
-                rescale(G);
-                G = 1.0f;
-            }
-            const float wg = __fdividef(sc.y, G);
-            uint64_t u[NC], aq[NC];
+#pragma unroll 1
+        for (int t = 0; t < nt; t += 4) { // four tokens' read-outs are reduced over the lanes together
+            float r[4 * NC], g[4];        // partial sums of this lane, token by token; decay scale of each token
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                const float x = wg * st.v[t][cl + c];
-                u[c] = f32x2(x, x);
-                aq[c] = 0ull;
-            }
-#pragma unroll
-            for (int m = 0; m < DM; ++m) {
-                const ulonglong2 kk = *reinterpret_cast<const ulonglong2 *>(&st.k[t][32 * m + 4 * part]);
-                const ulonglong2 qq = *reinterpret_cast<const ulonglong2 *>(&st.q[t][32 * m + 4 * part]);
+            for (int x = 0; x < 4; ++x) {
+                const bool valid = t + x < nt;
+                const float2 sc = *reinterpret_cast<const float2 *>(st.s[t + x]);
+                G *= valid ? sc.x : 1.0f;
+                if (G < 9.5367431640625e-7f) { // the same in every thread of the block
+                    rescale(G);
+                    G = 1.0f;
+                }
+                g[x] = G;
+                const float wg = valid ? __fdividef(sc.y, G) : 0.0f;
+                uint64_t u[NC], aq[NC];
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
-                    s[c][2 * m] = fma2(kk.x, u[c], s[c][2 * m]);
-                    s[c][2 * m + 1] = fma2(kk.y, u[c], s[c][2 * m + 1]);
-                    aq[c] = fma2(s[c][2 * m], qq.x, aq[c]);
-                    aq[c] = fma2(s[c][2 * m + 1], qq.y, aq[c]);
+                    const float y = wg * st.v[t + x][cl + c];
+                    u[c] = f32x2(y, y);
+                    aq[c] = 0ull;
+                }
+#pragma unroll
+                for (int m = 0; m < DM; ++m) {
+                    const ulonglong2 kk = *reinterpret_cast<const ulonglong2 *>(&st.k[t + x][32 * m + 4 * part]);
+                    const ulonglong2 qq = *reinterpret_cast<const ulonglong2 *>(&st.q[t + x][32 * m + 4 * part]);
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) {
+                        s[c][2 * m] = fma2(kk.x, u[c], s[c][2 * m]);
+                        s[c][2 * m + 1] = fma2(kk.y, u[c], s[c][2 * m + 1]);
+                        aq[c] = fma2(s[c][2 * m], qq.x, aq[c]);
+                        aq[c] = fma2(s[c][2 * m + 1], qq.y, aq[c]);
+                    }
+                }
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const float2 p2 = f32x2_parts(aq[c]);
+                    r[x * NC + c] = p2.x + p2.y;
                 }
             }
-            // reduction over the eight lanes of the group; with two columns the upper half of the lanes takes the second
-            float r[NC];
+            // transposing reduction over the eight lanes: value i of 4 NC ends in lane i (NC = 2) or lanes 2i, 2i + 1
+            int o = 4;
 #pragma unroll
-            for (int c = 0; c < NC; ++c) {
-                const float2 a = f32x2_parts(aq[c]);
-                r[c] = a.x + a.y;
+            for (int k = 2 * NC; k >= 1; k >>= 1, o >>= 1) {
+                const bool up = (lane & o) != 0;
+#pragma unroll
+                for (int i = 0; i < k; ++i) {
+                    const float send = up ? r[i] : r[i + k], keep = up ? r[i + k] : r[i];
+                    r[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
             }
-            const bool up = (lane & 4) != 0;
-            float v = NC == 2 ? (up ? r[NC - 1] : r[0]) : r[0];
-            v += __shfl_xor_sync(0xffffffffu, NC == 2 ? (up ? r[0] : r[NC - 1]) : r[0], 4);
-            v += __shfl_xor_sync(0xffffffffu, v, 2);
-            v += __shfl_xor_sync(0xffffffffu, v, 1);
-            const int c = NC == 2 && up ? 1 : 0;
-            if (!(lane & 3) && (NC == 2 || !up) && col + c < cols) {
-                const size_t at = (size_t)(row0 + t0 + t) * d.heads + h;
-                if (norm) gates[at].w = G * v * q_scale;
-                else heads_out[at * d.vdim_p + col + c] = G * v * q_scale;
+            if (NC == 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], 1);
+            const int x = part >> 1, c = NC == 2 ? part & 1 : 0;
+            const float v = (x < 2 ? (x == 0 ? g[0] : g[1]) : (x == 2 ? g[2] : g[3])) * q_scale * r[0];
+            if (t + x < nt && (NC == 2 || !(part & 1)) && col + c < cols) {
+                const size_t at = (size_t)(row0 + t0 + t + x) * d.heads + h;
+                float *dst = norm ? &gates[at].w : heads_out + at * d.vdim_p + col + c;
+                *dst = v;
             }
         }
         __syncthreads();
@@ -328,12 +355,12 @@ mlstm_out_kernel(MlstmDims d, const float *__restrict__ proj, int ldp, const flo
         const int j = lane * 4 + 128 * c;
         if (j >= d.vdim_p) continue;
         const float4 gg = __ldcs(reinterpret_cast<const float4 *>(g + j)), ww = __ldg(reinterpret_cast<const float4 *>(nw + j));
-        store_from_float(y + j, v[c].x * rn * ww.x * sigmoid_f(gg.x));
-        store_from_float(y + j + 1, v[c].y * rn * ww.y * sigmoid_f(gg.y));
-        store_from_float(y + j + 2, v[c].z * rn * ww.z * sigmoid_f(gg.z));
-        store_from_float(y + j + 3, v[c].w * rn * ww.w * sigmoid_f(gg.w));
+        store_from_float(y + j, v[c].x * rn * ww.x * gate_f(gg.x));
+        store_from_float(y + j + 1, v[c].y * rn * ww.y * gate_f(gg.y));
+        store_from_float(y + j + 2, v[c].z * rn * ww.z * gate_f(gg.z));
+        store_from_float(y + j + 3, v[c].w * rn * ww.w * gate_f(gg.w));
     }
-    for (int j = 256 + lane; j < d.vdim_p; j += 32) store_from_float(y + j, o[j] * inv * rn * nw[j] * sigmoid_f(g[j]));
+    for (int j = 256 + lane; j < d.vdim_p; j += 32) store_from_float(y + j, o[j] * inv * rn * nw[j] * gate_f(g[j]));
 }
 
 template <typename T>
@@ -370,7 +397,7 @@ int launch_mlstm_prompt(b200nn_ctx *ctx, const MlstmDims &d, bool b16, const flo
     if (sm.n_seq > 65535) return set_error(ctx, B200NN_ERR_SHAPE, "mlstm: too many sequences in a pass");
     if (ldp & 3) return set_error(ctx, B200NN_ERR_SHAPE, "mlstm: projection rows must keep 16-byte alignment");
     PREFER_SMEM_ONCE(mlstm_gate_kernel);
-    launch_pdl(ctx, mlstm_gate_kernel, dim3(d.heads, sm.n_seq), dim3(32), 0, d, proj, ldp, w, st, sm, (float4 *)gates);
+    launch_pdl(ctx, mlstm_gate_kernel, dim3(d.heads, sm.n_seq), dim3(256), 0, d, proj, ldp, w, st, sm, (float4 *)gates);
     CK_LAUNCH(ctx, "mlstm_gate_kernel");
     // columns per lane: two when that leaves every SM a dozen warps, else one
     const long long columns = (long long)d.vdim_p * d.heads * sm.n_seq;

@@ -427,9 +427,130 @@ def hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak):
     return out
 
 
+# --design zufilorn, beside a Vivezen of the same entry of HYBRID_SIZES: query / key columns of an attention map, inner size of
+# the two-step projections, residual streams
+ZUFILORN_SIZES = {"w1024": (64, 128, 2), "w2048": (64, 128, 2), "w4096": (64, 128, 4)}
+
+
+def zufilorn_kernels(reg, shape, own, batch, prompt, hbm_peak, tf_peak):
+    """The Zufilorn decoder's sequence kernels alone (see hybrid_kernels).  Prompt attention counts the visible (query, key)
+    pairs: per pair and head 2 maps x (2 dim + 2 vdim) flops; it also gives exponentials per second, the softmax's own
+    limit.  Recurrences count 4 dim vdim (mLSTM) and 7 dim vdim (delta rule with a decay per channel) flops per token and
+    head against the f32 FMA peak.  Decode counts the cache rows read or the states read and written, the stream update
+    the streams, the sublayer's output and the normalised row."""
+    import torch
+    from b200nn import ops
+    width, layers, vocab, H, KH, vdim, _, _, _, _, _ = shape
+    dim, rank, streams = own
+    stream = torch.cuda.ExternalStream(reg.stream)
+    dev, f32_peak, out = "cuda", 74.4, {}
+    B = max(1, min(batch, 16384 // prompt))
+    T = B * prompt
+    kw = 2 * dim + vdim
+    att = (H, KH, dim, vdim, 1024, dim ** -0.5, 30.0, 0.1, 0.5, 0.5, 1e-5)
+
+    def ints(*rows):
+        return torch.tensor([int(v) for r in rows for v in r], device=dev, dtype=torch.int32)
+
+    def measure(call, iters):
+        torch.cuda.synchronize()
+        call(0)
+        reg.synchronize()
+        return _graph_time(reg, stream, call, iters)
+
+    def by_bytes(name, us, nbytes):
+        out[name] = {"us": round(us, 1), "MB": round(nbytes / 1e6, 1), "GBps": round(nbytes / us / 1e3, 1),
+                     "frac_of_hbm_peak": round(nbytes / us / 1e3 / hbm_peak, 4)}
+
+    def by_f32(name, us, fl):
+        out[name] = {"tokens": T, "sequences": B, "us": round(us, 1), "tflops_f32": round(fl / us / 1e6, 2),
+                     "frac_of_f32_peak": round(fl / us / 1e6 / f32_peak, 4)}
+
+    r0 = [prompt * b for b in range(B)]
+    rpos, rslot = ints([i % prompt for i in range(T)]), ints([i // prompt for i in range(T)])
+    seq = ints(range(B), r0, [prompt] * B, [0] * B, [i // prompt for i in range(T)])
+    # attention, prompts
+    q = torch.randn(T, H * 2 * dim, device=dev).to(torch.bfloat16)
+    cache = torch.randn(B, KH, prompt, kw, device=dev).to(torch.bfloat16)
+    gate = torch.randn(max(T, 256), H, device=dev)
+    o = torch.empty(max(T, 256), H * vdim, device=dev, dtype=torch.bfloat16)
+    us = measure(lambda i: ops.diff_attention(att, q.data_ptr(), cache.data_ptr(), prompt, B, rpos.data_ptr(), rslot.data_ptr(), gate.data_ptr(), T,
+                                              o.data_ptr(), reg, B, prompt, seq.data_ptr()), 16)
+    pairs = B * H * prompt * (prompt + 1) // 2
+    fl = pairs * 2 * (2 * dim + 2 * vdim)
+    out["diff_prefill_tc_kernel"] = {"tokens": T, "us": round(us, 1), "tflops": round(fl / us / 1e6, 1),
+                                     "frac_of_bf16_peak": round(fl / us / 1e6 / tf_peak, 4), "Texp_per_s": round(2 * pairs / us / 1e6, 2)}
+    del cache
+    # attention, decoding after the prompt: the size's own batch, and 256 sequences where they fit
+    for nb in (batch, 256):
+        ctx = min(prompt, int(20e9 // (nb * KH * kw * 2)))
+        cap = ctx + 32
+        nbytes = nb * (KH * ctx * kw * 2 + H * (2 * dim + vdim) * 2)
+        copies = max(2, int(300e6 // (nb * KH * cap * kw * 2)) + 1)
+        caches = [torch.randn(nb, KH, cap, kw, device=dev, dtype=torch.bfloat16) for _ in range(copies)]
+        pos = ints([ctx - 1] * nb)
+        us = measure(lambda i: ops.diff_attention(att, q.data_ptr(), caches[i % copies].data_ptr(), cap, nb, pos.data_ptr(), None, gate.data_ptr(), nb,
+                                                  o.data_ptr(), reg), 6 * copies)
+        by_bytes(f"diff_decode_tc_kernel_rows{nb}_ctx{ctx}", us, nbytes)
+        del caches
+    # delta rule with a decay per channel
+    sh = (H, KH, vdim, vdim, 4, 1e-5)
+    cw, ext = 2 * KH * vdim + H * vdim, H * vdim
+    pw = -(-(cw + H) // 16) * 16
+    wts = [torch.randn(4, cw, device=dev), torch.full((H,), 0.1, device=dev), torch.zeros(H * vdim, device=dev), torch.ones(vdim, device=dev)]
+    ptrs = tuple(t.data_ptr() for t in wts)
+    rows = max(T, 256)
+    proj, ex = torch.randn(rows, pw, device=dev), torch.randn(rows, 2 * ext, device=dev)
+    conv, state = torch.zeros(256, 4, cw, device=dev), torch.zeros(B, H, vdim, vdim, device=dev)
+    scratch = torch.empty(T * (cw + H * vdim * 2 + H + KH + 4), device=dev)
+    us = measure(lambda i: ops.channel_delta_rule(sh, ptrs, proj.data_ptr(), ex.data_ptr(), conv.data_ptr(), state.data_ptr(), rpos.data_ptr(),
+                                                  rslot.data_ptr(), T, o.data_ptr(), reg, B, prompt, seq.data_ptr(), scratch.data_ptr()), 6)
+    by_f32("channel_delta_prompt", us, 7 * vdim * vdim * H * T)
+    for nb in (batch, 256):
+        copies = max(2, int(300e6 // (nb * H * vdim * vdim * 4)) + 1)
+        states = [torch.randn(nb, H, vdim, vdim, device=dev) * 0.01 for _ in range(copies)]
+        pos = ints([100] * nb)
+        us = measure(lambda i: ops.channel_delta_rule(sh, ptrs, proj.data_ptr(), ex.data_ptr(), conv.data_ptr(), states[i % copies].data_ptr(),
+                                                      pos.data_ptr(), None, nb, o.data_ptr(), reg), 6 * copies)
+        by_bytes(f"channel_delta_step_kernel_rows{nb}", us, nb * (2 * H * vdim * vdim * 4 + (pw + 2 * ext + 4 * cw) * 4 + H * vdim * 2))
+        del states
+    del proj, ex, scratch, conv
+    # mLSTM
+    sh = (H, vdim, vdim, 15.0, 1e-5)
+    pw = -(-(4 * H * vdim + 2 * H) // 4) * 4
+    wts = [torch.zeros(H, device=dev), torch.linspace(2, 6, H, device=dev), torch.ones(H, vdim, device=dev)]
+    ptrs = tuple(t.data_ptr() for t in wts)
+    proj, scratch = torch.randn(rows, pw, device=dev), torch.empty(T * H * (vdim + 4), device=dev)
+    nrm, mx = torch.zeros(256, H, vdim, device=dev), torch.zeros(256, H, device=dev)
+    us = measure(lambda i: ops.mlstm(sh, ptrs, proj.data_ptr(), state.data_ptr(), nrm.data_ptr(), mx.data_ptr(), rpos.data_ptr(), rslot.data_ptr(), T,
+                                     o.data_ptr(), reg, B, seq.data_ptr(), scratch.data_ptr()), 6)
+    by_f32("mlstm_prompt", us, 4 * vdim * vdim * H * T)
+    for nb in (batch, 256):
+        copies = max(2, int(300e6 // (nb * H * vdim * vdim * 4)) + 1)
+        states = [torch.randn(nb, H, vdim, vdim, device=dev) * 0.01 for _ in range(copies)]
+        pos = ints([100] * nb)
+        us = measure(lambda i: ops.mlstm(sh, ptrs, proj.data_ptr(), states[i % copies].data_ptr(), nrm.data_ptr(), mx.data_ptr(), pos.data_ptr(), None, nb,
+                                         o.data_ptr(), reg), 6 * copies)
+        by_bytes(f"mlstm_step_kernel_rows{nb}", us, nb * (2 * H * vdim * (vdim + 1) * 4 + pw * 4 + H * vdim * 2))
+        del states
+    del proj, scratch
+    # residual streams: update, next sublayer's input and norm
+    for nb in (T, batch):
+        copies = max(2, int(300e6 // (nb * streams * width * 4)) + 1)
+        xs = [torch.randn(nb, streams, width, device=dev) for _ in range(copies)]
+        y, ln, norm = torch.randn(nb, width, device=dev), torch.empty(nb, width, device=dev, dtype=torch.bfloat16), torch.ones(width, device=dev)
+        coef = torch.cat([torch.full((streams,), 1.0 / streams), torch.zeros(streams), torch.eye(streams).reshape(-1)]).to(dev)
+        us = measure(lambda i: ops.stream_step(nb, streams, width, xs[i % copies].data_ptr(), None, y.data_ptr(), coef.data_ptr(), coef.data_ptr(),
+                                               norm.data_ptr(), 1e-5, ln.data_ptr(), None, reg), 4 * copies)
+        by_bytes(f"stream_step_kernel_rows{nb}", us, nb * width * (2 * streams * 4 + 4 + 2))
+        del xs
+    return out
+
+
 def run_design(args):
-    """Prefill and decode throughput of the hybrid decoder beside a GPT-2 of the same width, depth, vocabulary and
-    batch (f32 family: fp16 tensor-core operands), N = 1, state resident, device-timed; not the headline."""
+    """Prefill and decode throughput of a model design beside the closest other model of the same width, depth, vocabulary
+    and batch, N = 1, state resident, device-timed; not the headline.  The hybrid decoder (vivezen) stands beside a GPT-2 of
+    the f32 family (fp16 tensor-core operands), zufilorn beside vivezen."""
     import torch
     import b200nn
     from b200nn import DecodeSession, Gpt2Config, Gpt2Model, LanguageModel, synth
@@ -469,7 +590,22 @@ def run_design(args):
         shape, batch, prompt, steps = HYBRID_SIZES[name]
         width, layers, vocab, H, KH, dim, rot, rank, qr, window, ff = shape
         rec = {"config": dict(zip(("width", "layers", "vocab", "heads", "kv_heads", "dim", "rot_dim", "kv_rank", "q_rank", "window", "ff"), shape)),
-               "sequences": batch, "prompt": prompt, "kernels": hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak)}
+               "sequences": batch, "prompt": prompt}
+        if args.design == "zufilorn":
+            rec["zufilorn"] = dict(zip(("map_dim", "rank", "streams"), ZUFILORN_SIZES[name]))
+            rec["zufilorn_kernels"] = zufilorn_kernels(reg, shape, ZUFILORN_SIZES[name], batch, prompt, hbm_peak, tf_peak)
+            reg.trim()
+        rec["kernels"] = hybrid_kernels(reg, shape, batch, prompt, hbm_peak, tf_peak)
+        if args.design == "zufilorn" and not args.kernels_only:
+            own = ZUFILORN_SIZES[name]
+            cfg = synth.zufilorn_config(width, layers, vocab, H, KH, own[0], dim, ff, prompt + 4 * steps + 8, own[2])
+            w = synth.zufilorn_weights(cfg, own[1])
+            m = LanguageModel.from_weights(cfg, w, reg)
+            rec["zufilorn_parameters"] = sum(a.size for a in w.values())
+            del w
+            rec["zufilorn_bf16"] = measure(m, batch, prompt, steps, vocab)
+            del m
+            reg.trim()
         if not args.kernels_only:
             cfg = synth.hybrid_config(width, layers, vocab, H, KH, dim, rot, rank, qr, window, ff)
             w = synth.hybrid_weights(cfg)
@@ -479,6 +615,7 @@ def run_design(args):
             rec["vivezen_bf16"] = measure(m, batch, prompt, steps, vocab)
             del m
             reg.trim()
+        if not args.kernels_only and args.design == "vivezen":
             g = Gpt2Config(layers, width, width // 64, vocab, prompt + 4 * steps + 8)
             gw = synth.gpt2_weights(g)
             rec["gpt2_parameters"] = sum(a.size for a in gw.values())
@@ -488,7 +625,7 @@ def run_design(args):
             del m
             reg.trim()
         line["sizes"][name] = rec
-    if not args.kernels_only:
+    if not args.kernels_only and args.design == "vivezen":
         line["gpt2_attention"] = attention_isolated(reg, hbm_peak, tf_peak)
     line["clocks"] = sampler.finish()
     print(json.dumps(line), flush=True)
@@ -778,8 +915,8 @@ def main():
     ap.add_argument("--cpu-steps", type=int, default=8)
     ap.add_argument("--cpu-prompt", type=int, default=32)
     ap.add_argument("--cpu-max-steps", type=int, default=64)
-    ap.add_argument("--design", default="", choices=["", "vivezen"],
-                    help="measure this model design at a few sizes beside a GPT-2 of equal width instead of the headline workload")
+    ap.add_argument("--design", default="", choices=["", "vivezen", "zufilorn"],
+                    help="measure this model design at a few sizes beside the closest other model of equal width instead of the headline workload")
     ap.add_argument("--sizes", default="", help="with --design: comma-separated subset of its sizes")
     ap.add_argument("--kernels-only", action="store_true", help="with --design: only the isolated kernels")
     args = ap.parse_args()
