@@ -22,9 +22,9 @@ __device__ __forceinline__ void store_cols(float *p, const float (&f)[V]) {
     *reinterpret_cast<typename Vec<V>::type *>(p) = *reinterpret_cast<const typename Vec<V>::type *>(f);
 }
 
-// S: streams at most; V: columns per access; NV: accesses per thread
-template <int S, int V, int NV, typename T>
-__global__ void __launch_bounds__(256)
+// S: streams at most; V: columns per access; NV: accesses per thread; NT: threads
+template <int S, int V, int NV, int NT, typename T>
+__global__ void __launch_bounds__(NT)
 stream_step_kernel(int n, int d, float *__restrict__ xs, const float *__restrict__ x0, const float *__restrict__ y, StreamCoef prev, StreamCoef next,
                    const float *__restrict__ norm, float eps, int ldo, T *__restrict__ out, float *__restrict__ x_sum) {
     __shared__ float red[32];
@@ -44,7 +44,7 @@ stream_step_kernel(int n, int d, float *__restrict__ xs, const float *__restrict
     float u[NV][V], sum = 0.0f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        const int c = (tid + i * 256) * V;
+        const int c = (tid + i * NT) * V;
 #pragma unroll
         for (int e = 0; e < V; ++e) u[i][e] = 0.0f;
         if (c >= d) continue;
@@ -90,7 +90,7 @@ stream_step_kernel(int n, int d, float *__restrict__ xs, const float *__restrict
     const float r = 1.0f / sqrtf(block_sum(sum, red) / (float)d + eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-        const int c = (tid + i * 256) * V;
+        const int c = (tid + i * NT) * V;
         if (c >= d) continue;
         float g[V];
         load_cols<V>(norm + c, g);
@@ -106,26 +106,29 @@ stream_step_kernel(int n, int d, float *__restrict__ xs, const float *__restrict
     }
 }
 
-template <int S, int V, int NV>
+template <int S, int V, int NV, int NT>
 void launch_s(b200nn_ctx *ctx, const StreamStep &a, bool b16) {
     if (b16) {
-        PREFER_SMEM_ONCE((stream_step_kernel<S, V, NV, __nv_bfloat16>));
-        launch_pdl(ctx, stream_step_kernel<S, V, NV, __nv_bfloat16>, dim3(a.rows), dim3(256), 0, a.n, a.d, a.xs, a.x0, a.y, a.prev, a.next, a.norm,
+        PREFER_SMEM_ONCE((stream_step_kernel<S, V, NV, NT, __nv_bfloat16>));
+        launch_pdl(ctx, stream_step_kernel<S, V, NV, NT, __nv_bfloat16>, dim3(a.rows), dim3(NT), 0, a.n, a.d, a.xs, a.x0, a.y, a.prev, a.next, a.norm,
                    a.eps, a.ldo, (__nv_bfloat16 *)a.out, a.x_sum);
     } else {
-        PREFER_SMEM_ONCE((stream_step_kernel<S, V, NV, float>));
-        launch_pdl(ctx, stream_step_kernel<S, V, NV, float>, dim3(a.rows), dim3(256), 0, a.n, a.d, a.xs, a.x0, a.y, a.prev, a.next, a.norm, a.eps,
+        PREFER_SMEM_ONCE((stream_step_kernel<S, V, NV, NT, float>));
+        launch_pdl(ctx, stream_step_kernel<S, V, NV, NT, float>, dim3(a.rows), dim3(NT), 0, a.n, a.d, a.xs, a.x0, a.y, a.prev, a.next, a.norm, a.eps,
                    a.ldo, (float *)a.out, a.x_sum);
     }
 }
 
 template <int S>
 void launch_v(b200nn_ctx *ctx, const StreamStep &a, bool b16) {
-    if (a.d % 4 || a.ldo % 4) launch_s<S, 1, 32>(ctx, a, b16);
-    else if (a.d <= 1024) launch_s<S, 4, 1>(ctx, a, b16);
-    else if (a.d <= 2048) launch_s<S, 4, 2>(ctx, a, b16);
-    else if (a.d <= 4096) launch_s<S, 4, 4>(ctx, a, b16);
-    else launch_s<S, 4, 8>(ctx, a, b16);
+    constexpr int WIDE = S <= 4 ? 1024 : 512; // threads per row of a decode step's few rows
+    if (a.d % 4 || a.ldo % 4) launch_s<S, 1, 32, 256>(ctx, a, b16);
+    else if (a.d <= 1024) launch_s<S, 4, 1, 256>(ctx, a, b16);
+    else if (a.rows <= ctx->sm_count && a.d <= 4 * WIDE) launch_s<S, 4, 1, WIDE>(ctx, a, b16);
+    else if (a.rows <= ctx->sm_count) launch_s<S, 4, 8192 / (4 * WIDE), WIDE>(ctx, a, b16);
+    else if (a.d <= 2048) launch_s<S, 4, 2, 256>(ctx, a, b16);
+    else if (a.d <= 4096) launch_s<S, 4, 4, 256>(ctx, a, b16);
+    else launch_s<S, 4, 8, 256>(ctx, a, b16);
 }
 
 }  // namespace

@@ -292,11 +292,12 @@ def test_sessions_and_sampling(reg):
 
 # ---- mechanisms alone ------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("rows", [7, 200])  # a decode step's and a prompt's block shapes
 @pytest.mark.parametrize("n,width", [(1, 24), (2, 90), (3, 1500), (4, 2052), (5, 64), (8, 4100), (2, 8192)])
-def test_stream_step(reg, n, width, dtype):
+def test_stream_step(reg, n, width, rows, dtype):
     import torch
     rng = np.random.default_rng(n + width)
-    rows, eps, flags = 7, 1e-4, 0 if dtype == "bfloat16" else b200nn.LM_F32
+    eps, flags = 1e-4, 0 if dtype == "bfloat16" else b200nn.LM_F32
     x0, y, norm = (rng.standard_normal(s).astype(np.float32) for s in ((rows, width), (rows, width), (width,)))
     c = [{"in": rng.standard_normal(n), "out": rng.standard_normal(n), "mix": rng.standard_normal((n, n))} for _ in range(2)]
     dc = [_dev(np.concatenate([v["in"], v["out"], v["mix"].reshape(-1)])) for v in c]
