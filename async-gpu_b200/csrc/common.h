@@ -76,7 +76,7 @@ struct b200nn_ctx {
     int int4_via_f16 = 1;         // int4 Linears with that many tiles dequantise the weight to fp16 once and use that GEMM
     std::shared_ptr<DevBuf> wh;   // the dequantised weight, [N,K] fp16, one Linear at a time
     int lm_portion = 0;           // hybrid models: most new tokens of one sequence in a pass (0 = 2048); read when a cache is created
-    int delta_cols = 0;           // state columns per lane of the delta-rule prompt kernel: 1 or 2 (0 = by the amount of work)
+    int delta_cols = 0;           // state columns per lane of the delta-rule and mLSTM prompt kernels: 1 or 2 (0 = by the amount of work)
     bool capturing = false;      // true while a decode step is being captured into a graph
     // one persistent kernel for all transformer blocks of an int4 decode step (decode_persistent.cu)
     int persist = 0;              // 1: decode steps of persist_min_rows..persist_max_rows rows take it (opt-in: measured

@@ -135,7 +135,8 @@ B200NN_API int32_t b200nn_ctx_set_gemv_max_rows(b200nn_ctx *ctx, int32_t rows);
  * (the residual GEMMs then need complete sums, i.e. cluster splits); sessions read it when created.
  * "lm_portion" (default 0 = 2048): most new tokens of one sequence a hybrid model's cache takes in a pass; a
  * windowed layer's ring holds the window plus this many rows.  Read when a cache or session is created.
- * "delta_cols" (default 0 = by the amount of work): state columns per lane of the delta rule's prompt kernel (1 or 2).
+ * "delta_cols" (default 0 = by the amount of work): state columns per lane of the prompt kernels of the delta rules and
+ * the mLSTM (1 or 2).
  * "persist" (default 0): decode steps of an int4 model run all transformer blocks as one cooperative
  * kernel (decode sessions whose shape it supports).  Measured slower than the per-op CUDA graph.
  * Its aids: "persist_min_rows" / "persist_max_rows" (batch range it is used for), "persist_prefetch_mb",
@@ -322,7 +323,7 @@ B200NN_API int32_t b200nn_gpt2_get_config(const b200nn_gpt2 *m, b200nn_gpt2_conf
 B200NN_API size_t b200nn_gpt2_quantized_memory_bytes(const b200nn_gpt2 *m);
 /* Read back the int4 data the model holds for one block Linear (which: 0 c_attn, 1 c_proj, 2 mlp.c_fc,
  * 3 mlp.c_proj; layer -1 with which 0 = the LM head), in the reference layout: packed [K/8,N], scales
- * [ceil(K/g),N] (already fp16-rounded).  Lets a checker run the same nibbles through its own math. */
+ * [ceil(K/g),N] (already fp16-rounded).  Lets a caller run the same nibbles through its own math. */
 B200NN_API int32_t b200nn_gpt2_get_int4(const b200nn_gpt2 *m, int32_t layer, int32_t which, uint32_t *packed,
                                         float *scales, size_t *k_out, size_t *n_out);
 

@@ -58,7 +58,7 @@ CONFIGS = {
     "delta": config(64, 101, 2, [layer(delta(4, 4, 64, 48, 3))]),
     "delta_taps1": config(40, 67, 1, [layer(delta(3, 1, 16, 36, 1), 33)]),
     "mlstm": config(72, 130, 4, [layer(mlstm(2, 64, 16, cap=20.0), 50)]),
-    "attention": config(48, 61, 2, [layer(attention(4, 4, 32, 64, every=1))]),
+    "attention": config(48, 61, 2, [layer(attention(3, 3, 48, 64, every=1))]),
     "attention_one_head": config(48, 61, 5, [layer(attention(1, 1, 36, 28, coef=0.0, diff=0.1), 21)]),
     # many query heads on one key / value head; sizes beyond the tensor-core kernels
     "group": config(96, 77, 2, [layer(attention(12, 1, 16, 32)), layer(attention(20, 1, 16, 16), 31)]),
@@ -457,7 +457,7 @@ def test_mlstm(reg, shape, cols):
         reg.set_tuning("delta_cols", 0)
 
 
-DIFF_SHAPES = [(4, 2, 32, 64, 0.3, 50.0), (2, 1, 64, 128, 0.5, 9.0), (3, 3, 128, 48, 0.0, 20.0), (2, 2, 96, 128, 0.7, 0.0), (12, 1, 48, 112, 0.3, 30.0),
+DIFF_SHAPES = [(6, 2, 32, 48, 0.35, 45.0), (2, 1, 64, 128, 0.5, 9.0), (3, 3, 128, 48, 0.0, 20.0), (2, 2, 96, 128, 0.7, 0.0), (12, 1, 48, 112, 0.3, 30.0),
                (20, 1, 16, 32, 0.2, 5.0), (2, 2, 160, 96, 0.4, 25.0), (4, 2, 64, 160, 0.6, 40.0)]
 
 
